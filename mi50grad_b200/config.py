@@ -273,6 +273,140 @@ def memory_budget(config: QwenConfig, max_seq_len: int = 2048, num_gpus: int = 1
     }
 
 
+# ---------------------------------------------------------------------------
+# Decoders whose layers are described one by one: a parallel mixer (windowed
+# attention beside a state-space recurrence) and a dense feed-forward, each with
+# a norm on its output only.
+# ---------------------------------------------------------------------------
+
+@dataclass(frozen=True)
+class WindowAttentionSpec:
+    """Sliding-window attention whose values are the keys as projected; Q and K
+    are normalised over the whole projection."""
+    heads: int
+    kv_heads: int
+    dim: int
+    rot_dims: int
+    rot_base: float
+    scale: float
+    window: int                       # 0: unlimited
+
+
+@dataclass(frozen=True)
+class SSDSpec:
+    """Mamba-2 recurrence: `heads` of size `vdim`, state size `state`, B and C
+    shared by the heads of a group, gated RMSNorm in `norm_groups` parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int                         # taps of the causal convolution
+    norm_groups: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
+class ParallelLayerSpec:
+    attention: WindowAttentionSpec
+    ssd: SSDSpec
+    left_scale: float
+    right_scale: float
+    ff: int = 0                       # 0: no feed-forward
+    weights_of: Optional[int] = None  # layer whose tensors this one uses
+
+
+@dataclass
+class DegedraConfig:
+    hidden_size: int
+    vocab_size: int
+    rms_norm_eps: float
+    layers: List[ParallelLayerSpec]
+    logit_softcap: float = 0.0        # 0: none
+
+    def __post_init__(self):
+        for i, l in enumerate(self.layers):
+            a, s = l.attention, l.ssd
+            if a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim or a.dim > 256:
+                raise ValueError(f"layer {i}: unsupported attention sizes {a}")
+            if s.heads % s.groups or s.inner % s.norm_groups or s.state > 256 or s.conv < 1:
+                raise ValueError(f"layer {i}: unsupported recurrence sizes {s}")
+            self.weight_layer(i)
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    def weight_layer(self, i: int) -> int:
+        """Index of the layer whose tensors layer i uses (itself, if it has its own)."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            seen.add(i)
+            i = self.layers[i].weights_of
+            if not 0 <= i < len(self.layers) or i in seen:
+                raise ValueError("weights_of does not lead to a layer with tensors")
+        return i
+
+    def cache_bytes(self, max_seq_len: int, batch: int = 1, elem: int = 2) -> int:
+        """K and V rows of every layer (head rows padded to 8 elements)."""
+        return sum(2 * batch * max_seq_len * l.attention.kv_heads * (-(-l.attention.dim // 8) * 8) * elem
+                   for l in self.layers)
+
+    def state_bytes(self, batch: int = 1, elem: int = 2) -> int:
+        return sum(batch * (l.ssd.heads * l.ssd.state * l.ssd.vdim * 4 + (l.ssd.conv - 1) * l.ssd.conv_channels * elem)
+                   for l in self.layers)
+
+
+def degedra_config_from_dict(c: dict) -> DegedraConfig:
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        if e.get("type") != "parallel":
+            raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
+        m = e["mixer"]
+        a, r = m["left"], m["right"]
+        if a.get("vdim", a["dim"]) != a["dim"]:
+            raise ValueError(f"layer {i}: the values are the projected keys, so vdim must equal dim")
+        mlp = e.get("mlp")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        layers.append(ParallelLayerSpec(
+            attention=WindowAttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["rot"]["dims"], float(a["rot"]["base"]),
+                                          float(a["scale"]), int((a.get("mask") or {}).get("size") or 0)),
+            ssd=SSDSpec(r["heads"], r["vdim"], r["state"], r["groups"], r["conv"], r["norm_groups"]),
+            left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]),
+            ff=0 if mlp is None else mlp["ff"], weights_of=e.get("weights_of")))
+    return DegedraConfig(hidden_size=c["width"], vocab_size=c["vocab"], rms_norm_eps=float(c["norm"]["eps"]),
+                         layers=layers, logit_softcap=float(c.get("logit_softcap") or 0.0))
+
+
+def degedra_config_to_dict(cfg: DegedraConfig) -> dict:
+    """The config.json form that `degedra_config_from_dict` reads."""
+    layers = []
+    for l in cfg.layers:
+        a, s = l.attention, l.ssd
+        e = {"type": "parallel",
+             "mixer": {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.dim, "scale": a.scale,
+                                "rot": {"base": a.rot_base, "dims": a.rot_dims}, "mask": {"size": a.window}},
+                       "right": {"heads": s.heads, "vdim": s.vdim, "state": s.state, "groups": s.groups, "conv": s.conv,
+                                 "norm_groups": s.norm_groups},
+                       "left_scale": l.left_scale, "right_scale": l.right_scale},
+             "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None}
+        if l.weights_of is not None:
+            e["weights_of"] = l.weights_of
+        layers.append(e)
+    out = {"architecture": "Degedra", "width": cfg.hidden_size, "vocab": cfg.vocab_size,
+           "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
+    if cfg.logit_softcap:
+        out["logit_softcap"] = cfg.logit_softcap
+    return out
+
+
 AR_MODES = ("exact", "deferred_ref", "deferred_consistent")
 
 

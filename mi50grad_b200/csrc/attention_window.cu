@@ -1,0 +1,505 @@
+// Sliding-window attention of a parallel mixer, and the preparation pass in front of both of its branches.
+//
+//   mix_prepare       RMSNorm of Q and of K over the WHOLE projection (all heads at once), rotation of the
+//                     first `rot` dimensions of every head in (i, i + rot/2) pairs, K and the values (K as
+//                     projected) into the cache, causal convolution + SiLU of the recurrence's inputs, its
+//                     step sizes.
+//   window decode     split-KV flash decoding, any head size up to 256, bf16 or fp32 cache.
+//   window rows       many query rows of one sequence: 64-row tiles on bf16 tensor cores (mma.sync) that
+//                     walk only the key blocks their windows reach.
+//
+// Visibility: the row at position p sees slots max(0, p - window + 1) .. p of its sequence (slot = position:
+// rows of a sequence are consecutive tokens, no draft trees).
+#include "mixers.cuh"
+
+// ---------------------------------------------------------------------------
+// prepare: grid (2 + convolution blocks, rows)
+// ---------------------------------------------------------------------------
+#define MP_THREADS 256
+#define MP_CONV 4                // channels per thread
+
+template <typename T>
+__global__ void __launch_bounds__(MP_THREADS) mix_prepare_kernel(const MixLayer L, const MixRun R) {
+    extern __shared__ float mp_v[];              // the projection part of one row
+    __shared__ float red[32];
+    pdl_launch_dependents();
+    const int r = blockIdx.y, part = blockIdx.x, tid = threadIdx.x;
+    const RowMeta rm = R.rows[r];
+    const T* row = (const T*)R.proj + (size_t)r * R.ld_proj;
+    if (part < 2) {
+        // ---- queries (part 0) or keys and values (part 1)
+        const int heads = part == 0 ? L.H : L.G, n = heads * L.d;
+        const T* src = row + (part == 0 ? L.off_q : L.off_k);
+        const float* nw = part == 0 ? L.q_norm : L.k_norm;
+        T* dst = part == 0 ? (T*)R.qbuf + (size_t)r * L.H * L.dp
+                           : (T*)L.kcache + ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
+        T* vdst = (T*)L.vcache + ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
+        pdl_wait();
+        float ss = 0.f;
+        for (int i = tid; i < n; i += MP_THREADS) { const float v = ld_f(src + i); mp_v[i] = v; ss += v * v; }
+        const float inv = rsqrtf(block_sum(ss, red) / (float)n + L.eps);      // (its barriers also publish mp_v)
+        const int half = L.rot >> 1;
+        const float* ct = L.cos_tab + (size_t)rm.pos * half;
+        const float* st = L.sin_tab + (size_t)rm.pos * half;
+        for (int i = tid; i < heads * L.dp; i += MP_THREADS) {
+            const int hd = i / L.dp, e = i % L.dp, j = hd * L.d + e;
+            float o = 0.f, raw = 0.f;
+            if (e < L.d) {
+                raw = mp_v[j];
+                o = raw * inv * nw[j];
+                if (e < L.rot) {
+                    const bool first = e < half;
+                    const int a = first ? e : e - half, jo = first ? j + half : j - half;
+                    const float other = mp_v[jo] * inv * nw[jo];
+                    o = first ? o * ct[a] - other * st[a] : o * ct[a] + other * st[a];
+                }
+            }
+            dst[i] = to_t<T>(o);
+            if (part == 1) vdst[i] = to_t<T>(raw);
+        }
+        return;
+    }
+    // ---- convolution over time of x | B | C, and (first block) the step sizes
+    const int C = L.heads * L.P + 2 * L.groups * L.N;
+    const T* hist = (const T*)L.conv_state + (size_t)rm.seq * (L.taps - 1) * C;
+    // rows of this sequence in front of r in this launch, as far as the taps reach
+    int local = 0;
+    while (local < L.taps - 1 && r - local - 1 >= 0 && R.rows[r - local - 1].seq == rm.seq) ++local;
+    pdl_wait();
+    if (part == 2 && tid < L.heads)
+        for (int h = tid; h < L.heads; h += MP_THREADS)
+            R.dtb[(size_t)r * R.ld_dt + h] = softplus_p(ld_f(row + L.off_dt + h) + L.dt_bias[h]);
+#pragma unroll
+    for (int u = 0; u < MP_CONV; ++u) {
+        const int c = ((part - 2) * MP_CONV + u) * MP_THREADS + tid;
+        if (c >= C) continue;
+        float a = L.conv_b[c];
+        for (int j = L.taps - 1; j >= 0; --j) {                 // j tokens back; oldest first
+            const float v = j <= local ? ld_f(row - (size_t)j * R.ld_proj + L.off_x + c)
+                                       : ld_f(hist + (size_t)(L.taps - 1 - (j - local)) * C + c);
+            a = fmaf(L.conv_w[(size_t)c * L.taps + (L.taps - 1 - j)], v, a);
+        }
+        ((T*)R.xbc)[(size_t)r * R.ld_xbc + c] = to_t<T>(silu_p(a));
+    }
+}
+
+B2_API int b2_mix_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (l->H < 1 || l->G < 1 || l->H % l->G || l->d > 256 || l->dp < l->d || (l->dp & 7) || l->rot > l->d || (l->rot & 1) ||
+        l->taps < 1 || l->groups < 1 || l->heads % l->groups)
+        return cudaErrorInvalidValue;
+    const int C = l->heads * l->P + 2 * l->groups * l->N;
+    dim3 grid(2 + (C + MP_THREADS * MP_CONV - 1) / (MP_THREADS * MP_CONV), r->n_rows);
+    const size_t smem = (size_t)(l->H > l->G ? l->H : l->G) * l->d * sizeof(float);
+    static SmemOptIn opt[2];
+    if (r->dt == DT_BF16) {
+        if (int e = opt[0].ensure((const void*)mix_prepare_kernel<bf16>, smem)) return e;
+        return launch_pdl(mix_prepare_kernel<bf16>, grid, dim3(MP_THREADS), smem, s, *l, *r);
+    }
+    if (int e = opt[1].ensure((const void*)mix_prepare_kernel<float>, smem)) return e;
+    return launch_pdl(mix_prepare_kernel<float>, grid, dim3(MP_THREADS), smem, s, *l, *r);
+}
+
+// ---------------------------------------------------------------------------
+// decode: grid (G * head blocks, rows, splits)
+// ---------------------------------------------------------------------------
+#define WD_WARPS 8
+#define WD_THREADS (WD_WARPS * 32)
+#define WD_GT 8                  // query heads per CTA
+#define WD_KEYS 4                // keys of a warp per soft-max update (and as many on their way)
+#define WD_MIN_SPLIT 64          // keys that are worth a CTA of their own
+#define WD_MAX_SPLITS 32
+
+// EPL consecutive elements of a cache row, as loaded
+template <typename T, int EPL> struct WRaw { uint32_t w[EPL * sizeof(T) / 4]; };
+template <typename T, int EPL>
+__device__ __forceinline__ void wr_load(WRaw<T, EPL>& v, const T* p, bool ok) {
+    constexpr int NW = EPL * sizeof(T) / 4;
+#pragma unroll
+    for (int i = 0; i < NW; ++i) v.w[i] = 0u;
+    if (!ok) return;
+    if constexpr (NW % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < NW / 4; ++i) {
+            const uint4 u = ((const uint4*)p)[i];
+            v.w[4 * i] = u.x; v.w[4 * i + 1] = u.y; v.w[4 * i + 2] = u.z; v.w[4 * i + 3] = u.w;
+        }
+    } else if constexpr (NW == 2) { const uint2 u = *(const uint2*)p; v.w[0] = u.x; v.w[1] = u.y; }
+    else v.w[0] = *(const uint32_t*)p;
+}
+template <typename T, int EPL>
+__device__ __forceinline__ float wr_get(const WRaw<T, EPL>& v, int e) {
+    if constexpr (sizeof(T) == 4) return __uint_as_float(v.w[e]);
+    else return __uint_as_float((e & 1) ? (v.w[e >> 1] & 0xffff0000u) : (v.w[e >> 1] << 16));
+}
+
+template <typename T, int EPL, int GT>
+__global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLayer L, const MixRun R) {
+    const int Gq = L.H / L.G, nhb = (Gq + GT - 1) / GT;
+    const int kvh = blockIdx.x / nhb, hb = (blockIdx.x % nhb) * GT, nh = min(GT, Gq - hb);
+    const int r = blockIdx.y, sp = blockIdx.z;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    pdl_launch_dependents();
+    const RowMeta rm = R.rows[r];
+    const int k1 = rm.pos + 1;                                               // keys [k0, k1)
+    const int k0 = L.window > 0 ? max(0, k1 - L.window) : 0;
+    const int total = k1 - k0;
+    const int nsplit = max(1, min(R.splits, (total + WD_MIN_SPLIT - 1) / WD_MIN_SPLIT));
+    if (sp >= nsplit) return;
+    const int per = (total + nsplit - 1) / nsplit;
+    const int a0 = k0 + sp * per, a1 = min(k1, a0 + per);
+    __shared__ float sm_m[WD_WARPS][GT], sm_l[WD_WARPS][GT], sm_f[WD_MAX_SPLITS][GT], sm_li[GT];
+    __shared__ float sm_acc[WD_WARPS][32 * EPL];
+    __shared__ int s_last;
+    pdl_wait();
+    const bool in = lane * EPL < L.dp;                       // dp is a multiple of EPL (<= 8): lanes are in or out as a whole
+    const int col = lane * EPL;
+    float q[GT][EPL], acc[GT][EPL], m[GT], l[GT];
+#pragma unroll
+    for (int h = 0; h < GT; ++h) {
+        m[h] = -INFINITY; l[h] = 0.f;
+        WRaw<T, EPL> qv;
+        wr_load(qv, (const T*)R.qbuf + ((size_t)r * L.H + kvh * Gq + hb + h) * L.dp + col, in && h < nh);
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) { q[h][e] = wr_get(qv, e) * L.attn_scale; acc[h][e] = 0.f; }
+    }
+    const size_t base = ((size_t)rm.seq * L.max_seq * L.G + kvh) * L.dp + col, stride = (size_t)L.G * L.dp;
+    const T* kc = (const T*)L.kcache + base;
+    const T* vc = (const T*)L.vcache + base;
+    WRaw<T, EPL> kn[WD_KEYS], vn[WD_KEYS];
+    auto fetch = [&](int s) {
+#pragma unroll
+        for (int i = 0; i < WD_KEYS; ++i) {
+            const int key = s + i * WD_WARPS + warp;
+            const bool ok = in && key < a1;
+            wr_load(kn[i], kc + (size_t)key * stride, ok);
+            wr_load(vn[i], vc + (size_t)key * stride, ok);
+        }
+    };
+    if (a0 < a1) fetch(a0);
+    for (int s = a0; s + warp < a1; s += WD_WARPS * WD_KEYS) {
+        WRaw<T, EPL> kk[WD_KEYS], vv[WD_KEYS];
+#pragma unroll
+        for (int i = 0; i < WD_KEYS; ++i) { kk[i] = kn[i]; vv[i] = vn[i]; }
+        if (s + WD_WARPS * WD_KEYS < a1) fetch(s + WD_WARPS * WD_KEYS);
+        float d[WD_KEYS][GT];
+#pragma unroll
+        for (int i = 0; i < WD_KEYS; ++i)
+#pragma unroll
+            for (int h = 0; h < GT; ++h) {
+                float x = 0.f;
+#pragma unroll
+                for (int e = 0; e < EPL; ++e) x = fmaf(q[h][e], wr_get(kk[i], e), x);
+                d[i][h] = x;
+            }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < WD_KEYS; ++i)
+#pragma unroll
+                for (int h = 0; h < GT; ++h) d[i][h] += __shfl_xor_sync(0xffffffffu, d[i][h], o);
+#pragma unroll
+        for (int h = 0; h < GT; ++h) {
+            float mn = m[h];
+#pragma unroll
+            for (int i = 0; i < WD_KEYS; ++i) if (s + i * WD_WARPS + warp < a1) mn = fmaxf(mn, d[i][h]);
+            const float corr = expf(m[h] - mn);              // (the first key of the pass is always inside: mn is finite)
+            float ps = 0.f, pw[WD_KEYS];
+#pragma unroll
+            for (int i = 0; i < WD_KEYS; ++i) { pw[i] = s + i * WD_WARPS + warp < a1 ? expf(d[i][h] - mn) : 0.f; ps += pw[i]; }
+            l[h] = l[h] * corr + ps;
+#pragma unroll
+            for (int e = 0; e < EPL; ++e) {
+                float a = acc[h][e] * corr;
+#pragma unroll
+                for (int i = 0; i < WD_KEYS; ++i) a = fmaf(pw[i], wr_get(vv[i], e), a);
+                acc[h][e] = a;
+            }
+            m[h] = mn;
+        }
+    }
+    // ---- merge the warps, one head at a time
+#pragma unroll
+    for (int h = 0; h < GT; ++h) if (lane == 0) { sm_m[warp][h] = m[h]; sm_l[warp][h] = l[h]; }
+    const int unit = (r * L.G + kvh) * nhb + (blockIdx.x % nhb);
+    float* my = R.attn_scratch + ((size_t)unit * R.splits + sp) * GT * (32 * EPL + 4);
+#pragma unroll
+    for (int h = 0; h < GT; ++h) {
+        if (h >= nh) break;
+        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) sm_acc[warp][col + e] = acc[h][e];
+        __syncthreads();
+        float mm = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < WD_WARPS; ++w) mm = fmaxf(mm, sm_m[w][h]);
+        float ll = 0.f, f[WD_WARPS];
+#pragma unroll
+        for (int w = 0; w < WD_WARPS; ++w) { f[w] = sm_m[w][h] == -INFINITY ? 0.f : expf(sm_m[w][h] - mm); ll += sm_l[w][h] * f[w]; }
+        for (int c = tid; c < L.d; c += WD_THREADS) {
+            float a = 0.f;
+#pragma unroll
+            for (int w = 0; w < WD_WARPS; ++w) a += sm_acc[w][c] * f[w];
+            if (nsplit == 1) ((T*)R.out)[(size_t)r * R.ldo + (kvh * Gq + hb + h) * L.d + c] = to_t<T>(a / ll * L.left_scale);
+            else {
+                my[h * (32 * EPL + 4) + c] = a;
+                if (c == 0) { my[h * (32 * EPL + 4) + 32 * EPL] = mm; my[h * (32 * EPL + 4) + 32 * EPL + 1] = ll; }
+            }
+        }
+    }
+    if (nsplit == 1) return;
+    // ---- merge the slices: the last CTA of this (row, key head, head block)
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        const int old = atomicAdd(&R.attn_counters[unit], 1);
+        s_last = old == nsplit - 1;
+        if (s_last) R.attn_counters[unit] = 0;
+        __threadfence();
+    }
+    __syncthreads();
+    if (!s_last) return;
+    const float* all = R.attn_scratch + (size_t)unit * R.splits * GT * (32 * EPL + 4);
+    if (tid < nh) {
+        const float* e0 = all + tid * (32 * EPL + 4) + 32 * EPL;
+        const size_t st = (size_t)GT * (32 * EPL + 4);
+        float mv[WD_MAX_SPLITS], lv[WD_MAX_SPLITS], mm = -INFINITY, ll = 0.f;
+#pragma unroll
+        for (int x = 0; x < WD_MAX_SPLITS; ++x) {
+            mv[x] = x < nsplit ? __ldcg(e0 + x * st) : -INFINITY;
+            lv[x] = x < nsplit ? __ldcg(e0 + x * st + 1) : 0.f;
+        }
+#pragma unroll
+        for (int x = 0; x < WD_MAX_SPLITS; ++x) mm = fmaxf(mm, mv[x]);
+#pragma unroll
+        for (int x = 0; x < WD_MAX_SPLITS; ++x) {
+            const float f = mv[x] == -INFINITY ? 0.f : expf(mv[x] - mm);
+            ll += lv[x] * f;
+            sm_f[x][tid] = f;
+        }
+        sm_li[tid] = 1.f / ll;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * L.d; i += WD_THREADS) {
+        const int h = i / L.d, c = i % L.d;
+        float a = 0.f;
+        for (int x0 = 0; x0 < nsplit; x0 += 8) {
+            float v[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                v[u] = x0 + u < nsplit ? __ldcg(all + ((size_t)(x0 + u) * GT + h) * (32 * EPL + 4) + c) : 0.f;
+#pragma unroll
+            for (int u = 0; u < 8; ++u) if (x0 + u < nsplit) a = fmaf(v[u], sm_f[x0 + u][h], a);
+        }
+        ((T*)R.out)[(size_t)r * R.ldo + (kvh * Gq + hb + h) * L.d + c] = to_t<T>(a * sm_li[h] * L.left_scale);
+    }
+}
+
+// floats of scratch for `rows` rows (attn_counters: rows * G * ceil(H / G / WD_GT) ints)
+B2_API long long b2_window_attn_scratch(int H, int G, int dp, int rows, int splits) {
+    const int nhb = (H / G + WD_GT - 1) / WD_GT, epl = dp <= 64 ? 2 : dp <= 128 ? 4 : 8;
+    return (long long)rows * G * nhb * splits * WD_GT * (32 * epl + 4);
+}
+B2_API int b2_window_attn_units(int H, int G, int rows) { return rows * G * ((H / G + WD_GT - 1) / WD_GT); }
+
+template <typename T, int EPL>
+static int launch_wd(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    const int Gq = l->H / l->G;
+    // (a smaller head block keeps fewer registers; scratch is laid out for at most WD_GT heads per block)
+    if (Gq <= 1) return launch_pdl(window_decode_kernel<T, EPL, 1>, dim3(l->G, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);
+    if (Gq <= 2) return launch_pdl(window_decode_kernel<T, EPL, 2>, dim3(l->G, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);
+    if (Gq <= 4) return launch_pdl(window_decode_kernel<T, EPL, 4>, dim3(l->G, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);
+    const int nhb = (Gq + WD_GT - 1) / WD_GT;
+    return launch_pdl(window_decode_kernel<T, EPL, WD_GT>, dim3(l->G * nhb, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);
+}
+template <typename T>
+static int launch_wd_t(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (l->dp <= 64) return launch_wd<T, 2>(l, r, s);
+    if (l->dp <= 128) return launch_wd<T, 4>(l, r, s);
+    return launch_wd<T, 8>(l, r, s);
+}
+B2_API int b2_window_attn_decode(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (l->dp > 256 || (l->dp & 7) || l->H % l->G || r->splits < 1 || r->splits > WD_MAX_SPLITS) return cudaErrorInvalidValue;
+    return r->dt == DT_BF16 ? launch_wd_t<bf16>(l, r, s) : launch_wd_t<float>(l, r, s);
+}
+
+// ---------------------------------------------------------------------------
+// many rows of ONE sequence, bf16: grid (64-row tiles, H), four warps of 16 rows
+// ---------------------------------------------------------------------------
+#define WR_ROWS 64
+#define WR_KEYS 64
+#define WR_PAD 8
+
+__device__ __forceinline__ void wr_ldsm4(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void wr_ldsm4_t(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void wr_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t wr_pack(float x, float y) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    return *(const uint32_t*)&h;
+}
+
+template <int DP>
+__global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, const MixRun R) {
+    constexpr int LD = DP + WR_PAD, NT_O = DP / 8, PPR = DP / 8;
+    extern __shared__ __align__(16) unsigned char wrs[];
+    bf16* Qs = (bf16*)wrs;                       // [64][LD]
+    bf16* Kb = Qs + WR_ROWS * LD;                // [2][64][LD]
+    bf16* Vb = Kb + 2 * WR_KEYS * LD;            // [2][64][LD]
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int row0 = blockIdx.x * WR_ROWS, nrows = min(WR_ROWS, R.n_rows - row0), head = blockIdx.y;
+    const int kvh = head / (L.H / L.G);
+    const RowMeta rm = R.rows[row0];
+    const int p0 = rm.pos;                       // positions of the tile: p0 .. p0 + nrows - 1
+    const int k_lo = L.window > 0 ? max(0, p0 - L.window + 1) : 0, k_hi = p0 + nrows;
+    const int b0 = k_lo / WR_KEYS, b1 = (k_hi + WR_KEYS - 1) / WR_KEYS;
+    const size_t kv_base = ((size_t)rm.seq * L.max_seq * L.G + kvh) * L.dp, kv_stride = (size_t)L.G * L.dp;
+    pdl_wait();
+    for (int i = tid; i < WR_ROWS * PPR; i += 128) {
+        const int pc = i % PPR, r = i / PPR;
+        bf16* dst = Qs + r * LD + pc * 8;
+        if (r < nrows && pc * 8 < L.dp) cp_async16(dst, (const bf16*)R.qbuf + ((size_t)(row0 + r) * L.H + head) * L.dp + pc * 8);
+        else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
+    }
+    auto stage = [&](int blk, int buf) {
+        for (int i = tid; i < WR_KEYS * PPR; i += 128) {
+            const int pc = i % PPR, r = i / PPR, slot = blk * WR_KEYS + r;
+            bf16* kd = Kb + (buf * WR_KEYS + r) * LD + pc * 8;
+            bf16* vd = Vb + (buf * WR_KEYS + r) * LD + pc * 8;
+            if (slot < k_hi && pc * 8 < L.dp) {
+                cp_async16(kd, (const bf16*)L.kcache + kv_base + (size_t)slot * kv_stride + pc * 8);
+                cp_async16(vd, (const bf16*)L.vcache + kv_base + (size_t)slot * kv_stride + pc * 8);
+            } else {
+                *(uint4*)kd = make_uint4(0u, 0u, 0u, 0u);
+                *(uint4*)vd = make_uint4(0u, 0u, 0u, 0u);
+            }
+        }
+    };
+    stage(b0, 0);
+    cp_async_commit();
+    float o[NT_O][4];
+#pragma unroll
+    for (int n = 0; n < NT_O; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    const bf16* qw = Qs + warp * 16 * LD;
+    const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
+    const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;
+    const float sc = L.attn_scale * 1.44269504f;             // scores in the log2 domain
+    const int q_lo = p0 + warp * 16 + g, q_hi = q_lo + 8;    // positions of this thread's two rows
+    const int w_lo = L.window > 0 ? q_lo - L.window : -1, w_hi = L.window > 0 ? q_hi - L.window : -1;     // last invisible slots
+    const int wp0 = p0 + warp * 16;                          // the warp's positions: wp0 .. wp0 + 15
+    for (int blk = b0; blk < b1; ++blk) {
+        const int buf = (blk - b0) & 1, s_base = blk * WR_KEYS;
+        cp_async_wait<0>();
+        __syncthreads();
+        if (blk + 1 < b1) stage(blk + 1, buf ^ 1);
+        cp_async_commit();
+        // nothing of this block is visible to the warp's rows
+        if (s_base > wp0 + 15 || (L.window > 0 && s_base + WR_KEYS - 1 <= wp0 - L.window) || warp * 16 >= nrows) continue;
+        const bf16* Kt = Kb + buf * WR_KEYS * LD;
+        const bf16* Vt = Vb + buf * WR_KEYS * LD;
+        float s[WR_KEYS / 8][4];
+#pragma unroll
+        for (int n = 0; n < WR_KEYS / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+#pragma unroll 4
+        for (int k0 = 0; k0 < DP; k0 += 16) {
+            uint32_t a[4];
+            wr_ldsm4(a, qw + a_row * LD + k0 + a_col);
+#pragma unroll
+            for (int np = 0; np < WR_KEYS / 16; ++np) {
+                uint32_t b[4];
+                wr_ldsm4(b, Kt + (np * 16 + b_row) * LD + k0 + b_col);
+                wr_mma(s[2 * np], a, b[0], b[1]);
+                wr_mma(s[2 * np + 1], a, b[2], b[3]);
+            }
+        }
+        float mx_lo = -INFINITY, mx_hi = -INFINITY;
+        const bool whole = s_base + WR_KEYS - 1 <= wp0 && (L.window <= 0 || s_base > wp0 + 15 - L.window);
+#pragma unroll
+        for (int n = 0; n < WR_KEYS / 8; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float v = s[n][e] * sc;
+                if (!whole) {
+                    const int slot = s_base + 8 * n + 2 * t + (e & 1);
+                    const bool vis = e >= 2 ? (slot <= q_hi && slot > w_hi) : (slot <= q_lo && slot > w_lo);
+                    if (!vis) v = -INFINITY;
+                }
+                s[n][e] = v;
+                if (e >= 2) mx_hi = fmaxf(mx_hi, v); else mx_lo = fmaxf(mx_lo, v);
+            }
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1)); mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1)); mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+        const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
+        const float rf_lo = mn_lo == -INFINITY ? 0.f : mn_lo, rf_hi = mn_hi == -INFINITY ? 0.f : mn_hi;
+        const float c_lo = exp2f(m_lo - rf_lo), c_hi = exp2f(m_hi - rf_hi);
+        m_lo = mn_lo; m_hi = mn_hi;
+        float rs_lo = 0.f, rs_hi = 0.f;
+        uint32_t pa[WR_KEYS / 16][4];
+#pragma unroll
+        for (int n = 0; n < WR_KEYS / 8; ++n) {
+            const float e0 = exp2f(s[n][0] - rf_lo), e1 = exp2f(s[n][1] - rf_lo);
+            const float e2 = exp2f(s[n][2] - rf_hi), e3 = exp2f(s[n][3] - rf_hi);
+            rs_lo += e0 + e1; rs_hi += e2 + e3;
+            pa[n >> 1][(n & 1) * 2 + 0] = wr_pack(e0, e1);
+            pa[n >> 1][(n & 1) * 2 + 1] = wr_pack(e2, e3);
+        }
+        l_lo = l_lo * c_lo + rs_lo; l_hi = l_hi * c_hi + rs_hi;
+#pragma unroll
+        for (int n = 0; n < NT_O; ++n) { o[n][0] *= c_lo; o[n][1] *= c_lo; o[n][2] *= c_hi; o[n][3] *= c_hi; }
+#pragma unroll
+        for (int k16 = 0; k16 < WR_KEYS / 16; ++k16)
+#pragma unroll
+            for (int np = 0; np < NT_O / 2; ++np) {
+                uint32_t b[4];
+                wr_ldsm4_t(b, Vt + (k16 * 16 + a_row) * LD + np * 16 + a_col);
+                wr_mma(o[2 * np], pa[k16], b[0], b[1]);
+                wr_mma(o[2 * np + 1], pa[k16], b[2], b[3]);
+            }
+    }
+    cp_async_wait<0>();
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int rr = warp * 16 + g + 8 * half;
+        if (rr >= nrows) continue;
+        const float f = L.left_scale / (half ? l_hi : l_lo);
+        bf16* dst = (bf16*)R.out + (size_t)(row0 + rr) * R.ldo + (size_t)head * L.d;
+#pragma unroll
+        for (int n = 0; n < NT_O; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int c = 8 * n + 2 * t + e;
+                if (c < L.d) dst[c] = __float2bfloat16(o[n][2 * half + e] * f);
+            }
+    }
+}
+
+template <int DP>
+static int launch_wr(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    const size_t smem = (size_t)(WR_ROWS + 4 * WR_KEYS) * (DP + WR_PAD) * sizeof(bf16);
+    static SmemOptIn opt;
+    if (int e = opt.ensure((const void*)window_rows_kernel<DP>, smem)) return e;
+    return launch_pdl(window_rows_kernel<DP>, dim3((r->n_rows + WR_ROWS - 1) / WR_ROWS, l->H), dim3(128), smem, s, *l, *r);
+}
+// All rows belong to one sequence, bf16 only (b2_window_attn_decode takes everything else).
+B2_API int b2_window_attn_rows(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (r->dt != DT_BF16 || r->n_seqs != 1 || l->dp > 256 || (l->dp & 7) || l->H % l->G) return cudaErrorInvalidValue;
+    if (l->dp <= 32) return launch_wr<32>(l, r, s);
+    if (l->dp <= 64) return launch_wr<64>(l, r, s);
+    if (l->dp <= 96) return launch_wr<96>(l, r, s);
+    if (l->dp <= 128) return launch_wr<128>(l, r, s);
+    return launch_wr<256>(l, r, s);
+}
+B2_API int b2_sizeof_mix_layer() { return (int)sizeof(MixLayer); }
+B2_API int b2_sizeof_mix_run() { return (int)sizeof(MixRun); }

@@ -21,10 +21,13 @@
 #include "kernels.cuh"
 #include "gemm_tc.cuh"
 #include "chain.cuh"
+#include "mixers.cuh"
 
 #define LIN_INT4 0
 #define LIN_F16 1
 #define LIN_NONE 2
+#define LIN_BF16 3
+#define LIN_F32 4
 
 struct LinearDesc {
     int kind;
@@ -108,6 +111,29 @@ struct ModelDesc {
     // INT8-activation FFN work buffers, sized for max(max_rows, max_prefill) rows
     void* q8_xq; float* q8_sx; void* q8_gate; void* q8_up; float* q8_down; void* q8_xn;
     CommCtx comm;
+    const struct MixerModelDesc* mixer;    // post-norm decoder of parallel mixers (csrc/mixers.cuh); null: the hybrid decoder above
+};
+
+// Post-norm decoders with dense bf16 / fp32 weights: x += norm1(mixer(x)), x += norm2(ff(x)).  The row, sequence,
+// logits and arg-max buffers are ModelDesc's; element-typed buffers (proj, attn_out, act, xn and the p_ forms)
+// hold bf16 or fp32 by `dt`.
+struct MixerLayerDesc {
+    MixLayer mix;
+    LinearDesc in_proj;           // [q | k | z | x | B | C | dt]
+    LinearDesc out_proj;          // [attention | recurrence] -> H
+    LinearDesc gate_up, down;     // kind LIN_NONE: no feed-forward
+    const float* norm1; const float* norm2;
+};
+struct MixerModelDesc {
+    const MixerLayerDesc* layers;
+    const float* final_norm;
+    float softcap; int dt;
+    int ss_np, ld_x;              // partial sums per row; row stride of p_xn
+    int ld_xbc, ld_dt, ld_u, ld_act, scratch_rows, pad;    // scratch_rows: rows the split-attention scratch holds
+    float* m; float* p_m;         // raw sublayer outputs [rows][H]
+    void* qbuf; void* xbc; float* dtb; float* ubuf;            // sized for max(max_rows, max_prefill) rows
+    float* attn_scratch; int* attn_counters; int* ssd_counters;
+    float* chunk_state; void* chunk_prev; float* chunk_decay;  // chunked scan (null: token by token only)
 };
 
 // Projections queued for one chain launch, with what the stand-alone GEMV path needs to run them
@@ -123,6 +149,8 @@ struct PendingChain {
 struct Driver {
     ModelDesc m;
     std::vector<LayerDesc> layers;
+    MixerModelDesc mx;                    // mlayers empty: not a mixer model
+    std::vector<MixerLayerDesc> mlayers;
     PendingChain pend;
     long long chain_launches = 0;         // chain kernels issued by the last step that was issued or captured
     long long exchanges = 0;              // cross-GPU exchanges of that step
@@ -159,6 +187,7 @@ static inline unsigned int* step_word(const ModelDesc& m) { return m.chain_count
 #define STEP_NO_COMMIT_DELTA 16 // DeltaNet state dry run
 #define STEP_MATERIALIZE_XN 32  // write the final-normed hidden states to xn (hidden-out interface)
 #define STEP_SPEC 64            // rows are draft trees: verify without touching the state, accept, commit
+#define STEP_HEAD_LAST 256      // many rows of one sequence: logits (and arg-max) of the last row only, in row 0 of the few-row buffers
 #define STEP_GEMM_PATH 128      // many rows: tensor-core GEMMs and the p_* buffers (else the GEMV path, <= 8 rows)
 
 #define CK(x) do { int e_ = (x); if (e_ != 0) return e_; } while (0)
@@ -356,6 +385,26 @@ static int spec_tail(Driver* d, const void* rows, const int* row_tokens, const i
     return 0;
 }
 
+// Arg-max over the logits of `rows` rows (many: the p_ buffers), then len += 1 of every sequence.
+static int argmax_advance(Driver* d, bool many, int rows, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    if (flags & STEP_ARGMAX) {
+        ArgmaxParams a;
+        memset(&a, 0, sizeof(a));
+        a.logits = many ? m.p_logits : m.logits; a.ld = m.ld_logits; a.n_rows = rows; a.vocab_local = m.vocab_local;
+        a.vocab_offset = m.vocab_offset; a.blocks = m.argmax_blocks; a.scratch = many ? m.p_argmax_scratch : m.argmax_scratch;
+        a.counters = many ? m.p_argmax_counters : m.argmax_counters; a.out_tokens = many ? m.p_out_tokens : m.out_tokens;
+        a.seqs = (flags & STEP_ADVANCE) ? (SeqState*)m.seqs : nullptr; a.rows = (const RowMeta*)(many ? m.p_rows : m.rows); a.comm = m.comm;
+        CK(b2_argmax(&a, s));
+        d->launches++;
+    }
+    if (flags & STEP_ADVANCE) {
+        CK(b2_advance(m.seqs, nullptr, n_seqs, 1, s));
+        d->launches++;
+    }
+    return 0;
+}
+
 static int step_impl(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
     const ModelDesc& m = d->m;
     if (rows < 1 || rows > m.max_rows || rows > B2_MAX_ROWS) return cudaErrorInvalidValue;
@@ -442,20 +491,7 @@ static int step_impl(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s)
         CK(b2_add_rmsnorm(m.h, nullptr, nullptr, last_norm, m.xn, nullptr, rows, m.H, m.eps, s));
         d->launches++;
     }
-    if (flags & STEP_ARGMAX) {
-        ArgmaxParams a;
-        memset(&a, 0, sizeof(a));
-        a.logits = m.logits; a.ld = m.ld_logits; a.n_rows = rows; a.vocab_local = m.vocab_local;
-        a.vocab_offset = m.vocab_offset; a.blocks = m.argmax_blocks; a.scratch = m.argmax_scratch;
-        a.counters = m.argmax_counters; a.out_tokens = m.out_tokens;
-        a.seqs = (flags & STEP_ADVANCE) ? (SeqState*)m.seqs : nullptr; a.rows = (const RowMeta*)m.rows; a.comm = m.comm;
-        CK(b2_argmax(&a, s));
-        d->launches++;
-    }
-    if (flags & STEP_ADVANCE) {
-        CK(b2_advance(m.seqs, nullptr, n_seqs, 1, s));
-        d->launches++;
-    }
+    CK(argmax_advance(d, false, rows, n_seqs, flags, s));
     if (flags & STEP_SPEC) {
         // without an arg-max this is a verify-only pass (hidden states out, nothing committed)
         if (flags & STEP_ADVANCE) return cudaErrorInvalidValue;
@@ -690,21 +726,8 @@ static int rows_impl(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
         CK(b2_gemm_f16_tc(&g, m.lm_head.w, m.lm_head.ldw, m.p_xn, m.H, s));
         d->launches++;
     }
-    if (flags & STEP_ARGMAX) {
-        if (!(flags & STEP_LM_HEAD)) return cudaErrorInvalidValue;
-        ArgmaxParams a;
-        memset(&a, 0, sizeof(a));
-        a.logits = m.p_logits; a.ld = m.ld_logits; a.n_rows = T; a.vocab_local = m.vocab_local;
-        a.vocab_offset = m.vocab_offset; a.blocks = m.argmax_blocks; a.scratch = m.p_argmax_scratch;
-        a.counters = m.p_argmax_counters; a.out_tokens = m.p_out_tokens;
-        a.seqs = (flags & STEP_ADVANCE) ? (SeqState*)m.seqs : nullptr; a.rows = (const RowMeta*)m.p_rows; a.comm = m.comm;
-        CK(b2_argmax(&a, s));
-        d->launches++;
-    }
-    if (flags & STEP_ADVANCE) {
-        CK(b2_advance(m.seqs, nullptr, n_seqs, 1, s));
-        d->launches++;
-    }
+    if ((flags & STEP_ARGMAX) && !(flags & STEP_LM_HEAD)) return cudaErrorInvalidValue;
+    CK(argmax_advance(d, true, T, n_seqs, flags, s));
     if (flags & STEP_SPEC) {
         if (flags & STEP_ADVANCE) return cudaErrorInvalidValue;
         if (flags & STEP_ARGMAX) CK(spec_tail(d, m.p_rows, m.p_row_tokens, m.p_out_tokens, n_seqs, s));
@@ -712,7 +735,173 @@ static int rows_impl(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
     return 0;
 }
 
+// ---------------------------------------------------------------------------
+// Post-norm decoders of parallel mixers.
+// ---------------------------------------------------------------------------
+// Decode projection; pn: the residual update its input still owes (x null), ss_out: partial sums for the next one.
+static int mixer_gemv(Driver* d, const LinearDesc& L, const void* x, int ldx, const PostNorm& pn, int rows, void* out, int ldo,
+                      int mode, float* ss_out, float softcap, cudaStream_t s) {
+    DenseGemvParams p;
+    memset(&p, 0, sizeof(p));
+    p.w = L.w; p.x = x; p.pn = pn; p.out = out; p.ss_out = ss_out; p.ldw = L.ldw; p.ldx = ldx; p.K = L.K; p.N = L.N;
+    p.rows = rows; p.ldo = ldo; p.mode = mode; p.dt = d->mx.dt; p.rpc = L.L; p.ss_np = d->mx.ss_np; p.softcap = softcap;
+    d->launches++;
+    return b2_gemv_dense(&p, s);
+}
+
+// Many-row projection: tcgen05 GEMM (bf16) or the fp32 GEMM.
+static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, int T, void* out, int ldo, int mode, float softcap,
+                      cudaStream_t s) {
+    d->launches++;
+    if (d->mx.dt == DT_F32) {
+        GemmF32Params p;
+        memset(&p, 0, sizeof(p));
+        p.w = (const float*)L.w; p.x = (const float*)x; p.out = out; p.ldw = L.ldw; p.ldx = ldx; p.K = L.K; p.N = L.N; p.T = T;
+        p.ldo = ldo; p.mode = mode; p.softcap = softcap;
+        return b2_gemm_f32(&p, s);
+    }
+    GemmTcParams p;
+    memset(&p, 0, sizeof(p));
+    const int ctas_n = (L.N + 127) / 128;
+    int tt = T >= 256 ? 256 : ((T + 15) & ~15);
+    if (ctas_n < 148) {                                    // few output tiles: cut the tokens until the grid fills one wave
+        int need = ((T + 148 / ctas_n - 1) / (148 / ctas_n) + 15) & ~15;
+        if (need < 64) need = 64;
+        if (need < tt) tt = need;
+    }
+    p.K = L.K; p.T = T; p.t_tile = tt; p.ldo = ldo; p.out = out; p.status = d->m.tc_status; p.bf16 = 1; p.softcap = softcap;
+    p.n_valid = mode == DG_SILU_PAIR ? L.N / 2 : L.N;
+    p.epi = mode == DG_SILU_PAIR ? TC_EPI_SILU_PAIR : (mode == DG_STORE ? TC_EPI_STORE_F16 : TC_EPI_STORE_F32);
+    return b2_gemm_f16_tc(&p, L.w, L.ldw, x, ldx, s);
+}
+
+static MixRun mixer_run(const Driver* d, bool many, int rows, int n_seqs, int flags) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    MixRun r;
+    memset(&r, 0, sizeof(r));
+    r.proj = many ? m.p_proj : m.proj; r.ld_proj = m.ld_proj; r.dt = x.dt;
+    r.rows = (const RowMeta*)(many ? m.p_rows : m.rows); r.seq_rows = m.seq_rows; r.n_rows = rows; r.n_seqs = n_seqs;
+    r.qbuf = x.qbuf; r.xbc = x.xbc; r.ld_xbc = x.ld_xbc; r.dtb = x.dtb; r.ld_dt = x.ld_dt; r.ubuf = x.ubuf; r.ld_u = x.ld_u;
+    r.splits = rows <= x.scratch_rows ? m.attn_splits : 1;
+    r.fuse_norm = rows == n_seqs || rows <= B2_MAX_ROWS;
+    r.out = many ? m.p_attn : m.attn_out; r.ldo = m.ld_attn; r.commit = (flags & STEP_NO_COMMIT_DELTA) ? 0 : 1;
+    r.attn_scratch = x.attn_scratch; r.attn_counters = x.attn_counters; r.ssd_counters = x.ssd_counters;
+    r.chunk_state = x.chunk_state; r.chunk_prev = x.chunk_prev; r.chunk_decay = x.chunk_decay;
+    return r;
+}
+
+struct LayerCount {
+    Driver* d; int li; long long l0;
+    LayerCount(Driver* d_, int li_) : d(d_), li(li_), l0(d_->launches) {}
+    ~LayerCount() { d->layer_launches[li] = (int)(d->launches - l0); }
+};
+
+// <= 8 rows.  The residual update of a sublayer is formed by the projection that follows it, so the stream
+// alternates between two buffers; the first is chosen so that it ends in m.h.
+static int mixer_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    if (rows < 1 || rows > m.max_rows || rows > B2_MAX_ROWS) return cudaErrorInvalidValue;
+    if (flags & STEP_SPEC) return cudaErrorNotSupported;
+    d->launches = 0; d->chain_launches = 0; d->exchanges = 0; d->pend.n = 0;
+    CK(b2_prepare_rows(m.rows_tmpl, m.seqs, m.rows, rows, nullptr, s)); d->launches++;
+    int flips = 0;
+    for (int li = 0; li < m.n_layers; ++li) flips += (li > 0) + (d->mlayers[li].down.kind != LIN_NONE);
+    float* h = (flips & 1) ? m.h_tmp : m.h;
+    float* h2 = (flips & 1) ? m.h : m.h_tmp;
+    if (flags & STEP_EMBED_TOKENS) {
+        CK(b2_embed_rows(m.embed, m.row_tokens, m.rows, m.seqs, h, nullptr, 0, rows, m.H, m.vocab, x.dt, s)); d->launches++;
+    } else {
+        // (an ordinary stream operation in any case: the kernels below read the row table ahead of their
+        // dependency wait, which is safe only if prepare_rows has completed before the first of them starts)
+        if (cudaError_t e = cudaMemcpyAsync(m.h_tmp, m.h, (size_t)rows * m.H * sizeof(float), cudaMemcpyDeviceToDevice, s)) return e;
+    }
+    const float* owed = nullptr;                 // weights of the norm whose residual update is still owed
+    int owed_np = 0;
+    PostNorm none;
+    memset(&none, 0, sizeof(none));
+    auto input = [&]() {
+        PostNorm pn;
+        memset(&pn, 0, sizeof(pn));
+        pn.h = h; pn.H = m.H; pn.eps = m.eps;
+        if (owed) { pn.m = x.m; pn.w = owed; pn.ss = m.ss; pn.np = owed_np; pn.hout = h2; }
+        return pn;
+    };
+    auto settled = [&]() { if (owed) { float* t = h; h = h2; h2 = t; } owed = nullptr; };
+    const MixRun r = mixer_run(d, false, rows, n_seqs, flags);
+    for (int li = 0; li < m.n_layers; ++li) {
+        const MixerLayerDesc& L = d->mlayers[li];
+        LayerCount count(d, li);
+        CK(mixer_gemv(d, L.in_proj, nullptr, 0, input(), rows, m.proj, m.ld_proj, DG_STORE, nullptr, 0.f, s));
+        settled();
+        CK(b2_mix_prepare(&L.mix, &r, s)); d->launches++;
+        CK(b2_window_attn_decode(&L.mix, &r, s)); d->launches++;
+        CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2;
+        CK(mixer_gemv(d, L.out_proj, m.attn_out, m.ld_attn, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
+        owed = L.norm1; owed_np = (m.H + L.out_proj.L - 1) / L.out_proj.L;
+        if (L.down.kind == LIN_NONE) continue;
+        CK(mixer_gemv(d, L.gate_up, nullptr, 0, input(), rows, m.act, x.ld_act, DG_SILU_PAIR, nullptr, 0.f, s));
+        settled();
+        CK(mixer_gemv(d, L.down, m.act, x.ld_act, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
+        owed = L.norm2; owed_np = (m.H + L.down.L - 1) / L.down.L;
+    }
+    // the last residual update and the final norm (xn feeds the head and the hidden-out interface)
+    CK(b2_post_norm(h, owed ? x.m : nullptr, owed, x.final_norm, m.xn, x.ld_x, rows, m.H, m.eps, x.dt, s)); d->launches++;
+    if (flags & STEP_LM_HEAD)
+        CK(mixer_gemv(d, m.lm_head, m.xn, x.ld_x, none, rows, m.logits, m.ld_logits, DG_STORE_F32, nullptr, x.softcap, s));
+    return argmax_advance(d, false, rows, n_seqs, flags, s);
+}
+
+static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    if (T < 1 || T > m.max_prefill) return cudaErrorInvalidValue;
+    if (flags & STEP_SPEC) return cudaErrorNotSupported;
+    d->launches = 0; d->chain_launches = 0; d->exchanges = 0;
+    CK(b2_prepare_rows(m.p_rows_tmpl, m.seqs, m.p_rows, T, nullptr, s)); d->launches++;
+    if (flags & STEP_EMBED_TOKENS)
+        CK(b2_embed_rows(m.embed, m.p_row_tokens, m.p_rows, m.seqs, m.p_h, m.p_xn, x.ld_x, T, m.H, m.vocab, x.dt, s));
+    else
+        CK(b2_post_norm(m.p_h, nullptr, nullptr, nullptr, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s));
+    d->launches++;
+    const MixRun r = mixer_run(d, true, T, n_seqs, flags);
+    const bool one = n_seqs == 1 && x.dt == DT_BF16;
+    for (int li = 0; li < m.n_layers; ++li) {
+        const MixerLayerDesc& L = d->mlayers[li];
+        LayerCount count(d, li);
+        const float* after = li + 1 == m.n_layers ? x.final_norm : nullptr;      // the last update also applies the final norm
+        CK(mixer_gemm(d, L.in_proj, m.p_xn, x.ld_x, T, m.p_proj, m.ld_proj, DG_STORE, 0.f, s));
+        CK(b2_mix_prepare(&L.mix, &r, s));
+        if (one && T >= 16) CK(b2_window_attn_rows(&L.mix, &r, s)); else CK(b2_window_attn_decode(&L.mix, &r, s));
+        d->launches += 2;
+        if (one && T >= 32 && x.chunk_state) { CK(b2_ssd_chunk(&L.mix, &r, s)); d->launches += 4; }
+        else { CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2; }
+        CK(mixer_gemm(d, L.out_proj, m.p_attn, m.ld_attn, T, x.p_m, m.H, DG_STORE_F32, 0.f, s));
+        const bool ff = L.down.kind != LIN_NONE;
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm1, ff ? nullptr : after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s)); d->launches++;
+        if (!ff) continue;
+        CK(mixer_gemm(d, L.gate_up, m.p_xn, x.ld_x, T, m.p_act, x.ld_act, DG_SILU_PAIR, 0.f, s));
+        CK(mixer_gemm(d, L.down, m.p_act, x.ld_act, T, x.p_m, m.H, DG_STORE_F32, 0.f, s));
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm2, after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s)); d->launches++;
+    }
+    if (flags & STEP_HEAD_LAST) {
+        if (n_seqs != 1 || (flags & STEP_ADVANCE)) return cudaErrorInvalidValue;
+        PostNorm none;
+        memset(&none, 0, sizeof(none));
+        const size_t off = (size_t)(T - 1) * x.ld_x * (x.dt == DT_BF16 ? 2 : 4);
+        CK(mixer_gemv(d, m.lm_head, (const char*)m.p_xn + off, x.ld_x, none, 1, m.logits, m.ld_logits, DG_STORE_F32, nullptr, x.softcap, s));
+        return argmax_advance(d, false, 1, 1, flags, s);
+    }
+    if (flags & STEP_LM_HEAD) {
+        if (T > m.p_logit_rows) return cudaErrorInvalidValue;
+        CK(mixer_gemm(d, m.lm_head, m.p_xn, x.ld_x, T, m.p_logits, m.ld_logits, DG_STORE_F32, x.softcap, s));
+    } else if (flags & STEP_ARGMAX) return cudaErrorInvalidValue;
+    return argmax_advance(d, true, T, n_seqs, flags, s);
+}
+
 static int run_impl(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
+    if (!d->mlayers.empty()) return (flags & STEP_GEMM_PATH) ? mixer_rows(d, rows, n_seqs, flags, s) : mixer_step(d, rows, n_seqs, flags, s);
     return (flags & STEP_GEMM_PATH) ? rows_impl(d, rows, n_seqs, flags, s) : step_impl(d, rows, n_seqs, flags, s);
 }
 
@@ -720,15 +909,19 @@ static int counted(Driver* d, int rc) {
     d->total_launches += d->launches; d->total_exchanges += d->exchanges;
     return rc;
 }
-B2_API int b2_driver_prefill(void* h, int T, int flags, cudaStream_t s) { return counted((Driver*)h, rows_impl((Driver*)h, T, 1, flags, s)); }
+B2_API int b2_driver_prefill(void* h, int T, int flags, cudaStream_t s) { return counted((Driver*)h, run_impl((Driver*)h, T, 1, flags | STEP_GEMM_PATH, s)); }
 B2_API int b2_driver_rows(void* h, int T, int n_seqs, int flags, cudaStream_t s) {
-    return counted((Driver*)h, rows_impl((Driver*)h, T, n_seqs, flags, s));
+    return counted((Driver*)h, run_impl((Driver*)h, T, n_seqs, flags | STEP_GEMM_PATH, s));
 }
 
 B2_API void* b2_driver_create(const ModelDesc* m, const LayerDesc* layers) {
     Driver* d = new Driver();
     d->m = *m;
-    d->layers.assign(layers, layers + m->n_layers);
+    memset(&d->mx, 0, sizeof(d->mx));
+    if (m->mixer) {
+        d->mx = *m->mixer;
+        d->mlayers.assign(m->mixer->layers, m->mixer->layers + m->n_layers);
+    } else d->layers.assign(layers, layers + m->n_layers);
     d->layer_launches.assign(m->n_layers, 0);
     // Off by default: measured on B200 (27B, one GPU, tg128) 213.6 tok/s with 4 blocks per warp, 213.1 with 2,
     // 208.7 with 8, against 213.9 without: the gaps between GEMVs are not waiting on HBM.
@@ -808,5 +1001,7 @@ B2_API int b2_driver_graph_nodes(void* h) {
 B2_API int b2_sizeof_linear_desc() { return (int)sizeof(LinearDesc); }
 B2_API int b2_sizeof_layer_desc() { return (int)sizeof(LayerDesc); }
 B2_API int b2_sizeof_model_desc() { return (int)sizeof(ModelDesc); }
+B2_API int b2_sizeof_mixer_layer_desc() { return (int)sizeof(MixerLayerDesc); }
+B2_API int b2_sizeof_mixer_model_desc() { return (int)sizeof(MixerModelDesc); }
 B2_API int b2_sizeof_row_meta() { return (int)sizeof(RowMeta); }
 B2_API int b2_sizeof_seq_state() { return (int)sizeof(SeqState); }

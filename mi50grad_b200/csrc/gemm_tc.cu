@@ -28,6 +28,7 @@
 // Every mbarrier wait is bounded; on expiry the kernel records a status, skips the rest of
 // its work, releases its tensor memory and returns.
 #include <cuda.h>
+#include <cuda_bf16.h>
 #include "kernels.cuh"
 #include "gemm_tc.cuh"
 #include "tc_util.cuh"
@@ -54,6 +55,12 @@ __device__ __forceinline__ uint32_t tc_nib_hi(uint32_t w) {
     uint32_t r;
     asm("lop3.b32 %0, %1, 0x00f000f0, 0x64006400, 0xea;" : "=r"(r) : "r"(w));
     return r;
+}
+
+// 16-bit output element in the operand type of the launch
+__device__ __forceinline__ void tc_store16(const GemmTcParams& p, size_t o, float v) {
+    if (p.bf16) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16(v);
+    else ((__half*)p.out)[o] = __float2half(v);
 }
 
 // PAIR: the kernel of CTA pairs is an instantiation of its own: a kernel that contains cta_group::2 instructions
@@ -243,7 +250,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                         float up = __shfl_down_sync(0xffffffffu, v, 8);
                         int tt = t0 + c0 + c;
                         if (is_gate && c0 + c < Tp && tt < p.T && o < p.n_valid)
-                            ((__half*)p.out)[(size_t)tt * p.ldo + o] = __float2half(silu_f(v) * up);
+                            tc_store16(p, (size_t)tt * p.ldo + o, silu_f(v) * up);
                     }
                 } else if (p.epi == TC_EPI_PUSH_F32) {
                     // plain stores into the owner's memory over NVLink (posted writes, 128 bytes per warp)
@@ -265,8 +272,8 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                         if (c0 + c < Tp && tt < p.T && n < p.n_valid) {
                             float v = __uint_as_float(r[c]);
                             size_t o = (size_t)tt * p.ldo + n;
-                            if (p.epi == TC_EPI_STORE_F16) ((__half*)p.out)[o] = __float2half(v);
-                            else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o] = v;
+                            if (p.epi == TC_EPI_STORE_F16) tc_store16(p, o, v);
+                            else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
                             else if (gridDim.z > 1) atomicAdd((float*)p.out + o, v);     // split-K partial
                             else ((float*)p.out)[o] += v;
                         }
@@ -309,7 +316,8 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
         {
             const bool dense = p.dense != 0;
             const int n1 = min(Tp, 256), n2 = Tp - n1;
-            const uint32_t idesc1 = make_idesc_f16(n1), idesc2 = make_idesc_f16(n2 > 0 ? n2 : 16);
+            const uint32_t fmt = p.bf16 ? TC_IDESC_BF16 : 0u;
+            const uint32_t idesc1 = make_idesc_f16(n1) | fmt, idesc2 = make_idesc_f16(n2 > 0 ? n2 : 16) | fmt;
             // descriptors differ between stages and k16 steps only in the start-address field (16-byte units)
             const uint64_t ad0 = make_desc_sw128(smem_u32(sA)), bd0 = make_desc_sw128(smem_u32(sB));
             const uint64_t a_step = (uint64_t)(a_bytes >> 4), b_step = (uint64_t)(b_stage_bytes >> 4), b_half = (256 * 128) >> 4;
@@ -390,6 +398,7 @@ B2_API size_t b2_gemm_tc_smem(int t_tile, int stages, int m_halves, int ring) {
 // x: [T][ldx] fp16 activations (ldx multiple of 8, base 16-byte aligned).
 static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w, const void* x, int ldx,
                      cudaStream_t stream) {
+    if (p->bf16 && !w) return cudaErrorInvalidValue;       // INT4 weights are dequantised to fp16
     if (p->T < 1 || p->t_tile < 16 || p->t_tile > 512 || (p->t_tile & 15) || (ldx & 7) || ((uintptr_t)x & 15))
         return cudaErrorInvalidValue;
     EncodeTiledFn enc = get_encode();
@@ -399,17 +408,18 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
     cuuint64_t strides[1] = {(cuuint64_t)ldx * 2};
     cuuint32_t box[2] = {TC_BK, 64};
     cuuint32_t estr[2] = {1, 1};
-    CUresult r = enc(&map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void*)x, dims, strides, box, estr,
+    const CUtensorMapDataType dtype = p->bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+    CUresult r = enc(&map, dtype, 2, (void*)x, dims, strides, box, estr,
                      CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                      CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return cudaErrorInvalidValue;
     CUtensorMap wmap = map;
     if (w) {
-        if ((ldw & 7) || ((uintptr_t)w & 15) || (p->K % TC_BK)) return cudaErrorInvalidValue;
+        if ((ldw & 7) || ((uintptr_t)w & 15)) return cudaErrorInvalidValue;
         cuuint64_t wd[2] = {(cuuint64_t)p->K, (cuuint64_t)n_rows_w};
         cuuint64_t ws[1] = {(cuuint64_t)ldw * 2};
         cuuint32_t wb[2] = {TC_BK, TC_BM};
-        r = enc(&wmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void*)w, wd, ws, wb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+        r = enc(&wmap, dtype, 2, (void*)w, wd, ws, wb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                 CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) return cudaErrorInvalidValue;
     }
@@ -425,11 +435,11 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
     size_t per_stage = (size_t)q.m_halves * TC_A_BYTES + (size_t)((q.t_tile + 63) / 64) * 64 * 128 / (q.cta_pair ? 2 : 1);
     // as many stages as shared memory holds next to the weight ring, an even number (the two producer
     // groups alternate stages); deep pipelines matter most for few tokens, where a stage is consumed quickly
-    const int ring = TC_RING_OF(q.cta_pair != 0);
+    const int ring = q.dense ? 0 : TC_RING_OF(q.cta_pair != 0);      // (dense weights need no ring of packed weights)
     const size_t fixed = 1024 + 256 + (size_t)ring * 2 * (TC_PRODUCERS * 32) * 16;
     int stages = (int)((227 * 1024 - fixed) / per_stage);
     stages = stages > 8 ? 8 : stages;
-    q.stages = stages < 2 ? 2 : (q.m_halves == 2 ? stages : (stages & ~1));
+    q.stages = stages < 2 ? 2 : (q.m_halves == 2 || q.dense ? stages : (stages & ~1));
     size_t smem = b2_gemm_tc_smem(q.cta_pair ? q.t_tile / 2 : q.t_tile, q.stages, q.m_halves, ring);
     static SmemOptIn optin;
     {
@@ -457,15 +467,16 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
 B2_API int b2_gemm_int4_tc(const GemmTcParams* p, const void* x, int ldx, cudaStream_t stream) {
     return launch_tc(p, nullptr, 0, 0, x, ldx, stream);
 }
-// Dense fp16 weights w[N][ldw] (row = output feature) take the same pipeline: the weight tile is a
+// Dense fp16 or bf16 (p->bf16) weights w[N][ldw] (row = output feature) take the same pipeline: the weight tile is a
 // second TMA load into the stage the dequantising warps would have filled.  p->K, T, t_tile, n_valid (= N),
 // ldo, epi, out, status are used; the INT4 fields are ignored.
 B2_API int b2_gemm_f16_tc(const GemmTcParams* p, const void* w, int ldw, const void* x, int ldx, cudaStream_t stream) {
     if (!w || p->n_valid < 1) return cudaErrorInvalidValue;
     GemmTcParams q = *p;
-    q.KB = q.K / TC_BK;
-    q.NTL = (q.n_valid + TC_BM - 1) / TC_BM * (TC_BM / 16);
+    q.KB = (q.K + TC_BK - 1) / TC_BK;        // a ragged last block is zero-filled by both TMA loads
+    const int n_rows_w = q.epi == TC_EPI_SILU_PAIR ? 2 * q.n_valid : q.n_valid;      // (gate / up rows interleaved by 8)
+    q.NTL = (n_rows_w + TC_BM - 1) / TC_BM * (TC_BM / 16);
     q.qfrag = nullptr; q.szfrag = nullptr;
-    return launch_tc(&q, w, ldw, q.n_valid, x, ldx, stream);
+    return launch_tc(&q, w, ldw, n_rows_w, x, ldx, stream);
 }
 B2_API int b2_sizeof_gemm_tc_params() { return (int)sizeof(GemmTcParams); }

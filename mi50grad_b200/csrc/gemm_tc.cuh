@@ -33,6 +33,8 @@ struct GemmTcParams {
                                  // products are added to out with atomic adds (0 or 1: no split)
     int cta_pair;                // 1: adjacent output tiles run as CTA pairs (cta_group::2 MMAs, M = 256 over two SMs); needs
                                  // 128-output CTAs, t_tile 256 or 512 dividing T, an even number of output tiles
+    int bf16;                // 1 (dense weights only): operands and 16-bit outputs are bf16 instead of fp16
+    float softcap;           // TC_EPI_STORE_F32: > 0 stores softcap * tanh(y / softcap)
     int pad3;
 };
 

@@ -150,6 +150,7 @@ __device__ __forceinline__ uint64_t make_desc_sw128(uint32_t smem_addr) {
     d |= (uint64_t)2 << 61;                                // SWIZZLE_128B
     return d;
 }
+#define TC_IDESC_BF16 ((1u << 7) | (1u << 10))      // both operands bf16 (or-ed into an fp16 descriptor)
 // Instruction descriptor: fp16 x fp16 -> fp32, both operands K-major, M = 128, N = n.
 __device__ __forceinline__ uint32_t make_idesc_f16(int n) {
     return (1u << 4) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);

@@ -111,6 +111,15 @@ class InferenceEngine:
         if quant_format not in ("w4a16", "w8a8", "w4a8"):
             raise ValueError("quant_format must be w4a16, w8a8 or w4a8")
         self.quant_format = quant_format
+        self.use_int4_attention = use_int4_attention
+        self._init_common(config, device_id, max_seq_len, tp_size, tp_rank, engine_config, comm, max_batch)
+        self.spec: ShardSpec = make_shard_spec(config, tp_size, tp_rank)
+        self.states = SequenceStates(config, self.spec, max_seq_len, max_batch, self.device)
+        self._init_rope_tables()
+
+    def _init_common(self, config, device_id: int, max_seq_len: int, tp_size: int, tp_rank: int,
+                     engine_config: Optional[EngineConfig], comm, max_batch: int):
+        """What an engine needs before its architecture matters."""
         self.config = config
         self.ecfg = (engine_config or EngineConfig()).replace(
             tp_size=tp_size, tp_rank=tp_rank, max_seq_len=max_seq_len, max_batch=max_batch)
@@ -118,16 +127,13 @@ class InferenceEngine:
         torch.cuda.set_device(self.device)
         self.lib = L.lib()
         self.tp_size, self.tp_rank = tp_size, tp_rank
-        self.spec: ShardSpec = make_shard_spec(config, tp_size, tp_rank)
         self.max_seq_len, self.max_batch = max_seq_len, max_batch
         self.max_rows = L.MAX_ROWS
         self.comm = comm
-        self.use_int4_attention = use_int4_attention
-        self.layers: List[Optional[DeviceLayer]] = [None] * config.num_hidden_layers
+        self.layers: List = [None] * config.num_hidden_layers
         self.embed: Optional[torch.Tensor] = None
         self.lm_head: Optional[DeviceLinear] = None
         self.final_norm: Optional[torch.Tensor] = None
-        self.states = SequenceStates(config, self.spec, max_seq_len, max_batch, self.device)
         self._driver = None
         self._exch_carry = 0
         self._graph_key = None
@@ -135,7 +141,6 @@ class InferenceEngine:
         self._ptmpl_key = None
         self._launch_counts: Dict[int, int] = {}
         self._steps = 0
-        self._init_rope_tables()
 
     # ------------------------------------------------------------------ set-up
     @property
@@ -302,6 +307,22 @@ class InferenceEngine:
         return self.weight_bytes()
 
     # ------------------------------------------------------------------ driver
+    def _work_allocator(self):
+        """alloc(shape, dtype) of zeroed work buffers; with debug_guards each one sits between poisoned
+        bands that are checked after every eager step (utils/guards.py)."""
+        self._guards = None
+        if self.ecfg.debug_guards:
+            from ..utils.guards import GuardedAllocator
+            self._guards = GuardedAllocator(self.device)
+        counter = [0]
+
+        def alloc(shape, dtype):
+            if self._guards is None:
+                return torch.zeros(*shape, dtype=dtype, device=self.device)
+            counter[0] += 1
+            return self._guards.zeros(f"#{counter[0]}", shape, dtype)
+        return alloc
+
     def _comm_ctx(self) -> L.CommCtx:
         if self.comm is not None and self.tp_size > 1:
             return self.comm.ctx()
@@ -316,19 +337,7 @@ class InferenceEngine:
         cfg, sp, dev, R = self.config, self.spec, self.device, self.max_rows
         H = cfg.hidden_size
         lins = [l for dl in self.layers for l in (dl.in_proj, dl.out_proj, dl.gate_up, dl.down)] + [self.lm_head]
-        # work buffers; with debug_guards each one sits between poisoned bands that are checked after
-        # every eager step (utils/guards.py)
-        self._guards = None
-        if self.ecfg.debug_guards:
-            from ..utils.guards import GuardedAllocator
-            self._guards = GuardedAllocator(dev)
-        counter = [0]
-
-        def alloc(shape, dtype):
-            if self._guards is None:
-                return torch.zeros(*shape, dtype=dtype, device=dev)
-            counter[0] += 1
-            return self._guards.zeros(f"#{counter[0]}", shape, dtype)
+        alloc = self._work_allocator()
         f32 = lambda *s: alloc(s, torch.float32)
         f16 = lambda *s: alloc(s, torch.float16)
         i32 = lambda *s: alloc(s, torch.int32)
@@ -633,6 +642,52 @@ class InferenceEngine:
         self.buf["h"][:1].copy_(self.buf["p_h"][n - 1:n])
         self.states.seqs[seq, 1] = tok[0]
         return int(tok[0].item())
+
+    def forward_tokens(self, tokens: Sequence[int], seq: int = 0, want: Sequence[int] = ()) -> torch.Tensor:
+        """Feed the next tokens of a sequence (any number, continuing from its cache and state) and return
+        the logits after the places `want` among them: fp32 [len(want), local vocabulary], device.  The
+        portion goes through the steps that serving uses: one token through the decode step (as
+        `step_host`), up to eight through the few-row step, more through the many-row path."""
+        self._ensure_driver()
+        tokens, want = [int(t) for t in tokens], [int(w) for w in want]
+        n, vl = len(tokens), self.spec.vocab_local
+        length = self.states.length(seq)
+        if n < 1 or any(not 0 <= w < n for w in want):
+            raise ValueError("no tokens, or a wanted place outside the portion")
+        if length + n > self.max_seq_len:
+            raise ValueError(f"{length} + {n} tokens exceed max_seq_len = {self.max_seq_len}")
+        if any(not 0 <= t < self.config.vocab_size for t in tokens):
+            raise ValueError("token id outside the vocabulary")
+        out = torch.empty(len(want), vl, dtype=torch.float32, device=self.device)
+
+        def keep(first, count, logits):
+            for j, w in enumerate(want):
+                if first <= w < first + count:
+                    out[j].copy_(logits[w - first, :vl])
+        if n == 1 and length > 0:
+            self.states.set_token(seq, tokens[0])
+            self.decode_tokens(1, [seq], collect=False)
+            keep(0, 1, self.buf["logits"])
+            return out
+        i = 0
+        while i < n:
+            rest = n - i
+            if rest <= self.max_rows or not self.use_tc_prefill:
+                c = min(rest, self.max_rows)
+                hit = any(i <= w < i + c for w in want)
+                self.step_tokens(tokens[i:i + c], seq, logits=hit)
+                keep(i, c, self.buf["logits"])
+            else:
+                c = min(rest, self.max_prefill)
+                hit = any(i <= w < i + c for w in want)
+                if hit:
+                    c = min(c, self.step_rows)
+                    hit = any(i <= w < i + c for w in want)
+                self.buf["p_row_tokens"][:c].copy_(torch.tensor(tokens[i:i + c], dtype=torch.int32).to(self.device))
+                self._prefill_rows(c, seq, L.STEP_EMBED_TOKENS | (L.STEP_LM_HEAD if hit else 0))
+                keep(i, c, self.buf["p_logits"])
+            i += c
+        return out
 
     def score_tokens(self, tokens: Sequence[int], seq: int = 0) -> torch.Tensor:
         """Teacher-forced log-probabilities: feeds `tokens` to an empty sequence slot and returns

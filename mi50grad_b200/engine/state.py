@@ -16,7 +16,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..config import QwenConfig
+from ..config import DegedraConfig, QwenConfig
 from ..parallel.sharding import ShardSpec
 
 DN_COLS = 32
@@ -79,15 +79,31 @@ class SequenceSnapshot:
     conv: torch.Tensor
 
 
-class SequenceStates:
-    """Lengths + caches of all slots.  `seqs` is the device array of
-    {len, token, pad, pad} the kernels read."""
+class SlotStates:
+    """Sequence slots: the device array `seqs` of {len, token, pad, pad} the kernels
+    read, and which slots are handed out."""
 
-    def __init__(self, cfg: QwenConfig, spec: ShardSpec, max_seq_len: int, max_batch: int, device):
-        self.kv = KVCache(cfg, spec, max_seq_len, max_batch, device)
-        self.dn = DeltaNetState(cfg, spec, max_batch, device)
+    def __init__(self, max_batch: int, device):
         self.seqs = torch.zeros(max_batch, 4, dtype=torch.int32, device=device)
         self.max_batch = max_batch
+        self._free = list(range(max_batch))
+
+    def acquire(self) -> int:
+        """A free slot, empty."""
+        if not self._free:
+            raise RuntimeError(f"all {self.max_batch} sequence slots are in use")
+        seq = self._free.pop(0)
+        self.reset(seq)
+        return seq
+
+    def release(self, seq: int):
+        """Give a slot back."""
+        if seq in self._free or not 0 <= seq < self.max_batch:
+            raise ValueError(f"slot {seq} is not in use")
+        self._free.insert(0, seq)
+
+    def reset(self, seq: Optional[int] = None):
+        raise NotImplementedError
 
     def lengths(self) -> List[int]:
         return self.seqs[:, 0].tolist()
@@ -103,6 +119,15 @@ class SequenceStates:
 
     def token(self, seq: int = 0) -> int:
         return int(self.seqs[seq, 1].item())
+
+
+class SequenceStates(SlotStates):
+    """Lengths + caches of all slots of the hybrid decoder."""
+
+    def __init__(self, cfg: QwenConfig, spec: ShardSpec, max_seq_len: int, max_batch: int, device):
+        super().__init__(max_batch, device)
+        self.kv = KVCache(cfg, spec, max_seq_len, max_batch, device)
+        self.dn = DeltaNetState(cfg, spec, max_batch, device)
 
     def reset(self, seq: Optional[int] = None):
         if seq is None:
@@ -144,3 +169,72 @@ class SequenceStates:
         dev = self.seqs.device
         self.restore(SequenceSnapshot(seq, int(sd["length"]), int(sd["token"]), sd["k"].to(dev),
                                       sd["v"].to(dev), sd["S"].to(dev), sd["conv"].to(dev)), seq)
+
+
+@dataclass
+class MixerSnapshot:
+    """Device copy of everything position-dependent for one slot of a `MixerStates`."""
+    seq: int
+    length: int
+    token: int
+    kv: Optional[List[tuple]]
+    state: List[tuple]
+
+
+class MixerStates(SlotStates):
+    """Slots of a decoder of parallel mixers.  Every layer has arrays of its own
+    (layers may differ in size, and a layer that shares another's weights still has
+    its own history): K and V rows [slot][max_seq][kv_heads][dim padded to 8] in the
+    element type, the recurrent state [slot][heads][state][vdim] in fp32, and the
+    convolution's last taps - 1 inputs [slot][taps-1][channels]."""
+
+    def __init__(self, cfg: DegedraConfig, max_seq_len: int, max_batch: int, device, dtype: torch.dtype):
+        super().__init__(max_batch, device)
+        self.max_seq_len = max_seq_len
+        z = lambda *sh, dt=dtype: torch.zeros(*sh, dtype=dt, device=device)
+        self.k, self.v, self.S, self.conv = [], [], [], []
+        for l in cfg.layers:
+            a, s = l.attention, l.ssd
+            dp = -(-a.dim // 8) * 8
+            self.k.append(z(max_batch, max_seq_len, a.kv_heads, dp))
+            self.v.append(z(max_batch, max_seq_len, a.kv_heads, dp))
+            self.S.append(z(max_batch, s.heads, s.state, s.vdim, dt=torch.float32))
+            self.conv.append(z(max_batch, s.conv - 1, s.conv_channels))
+
+    def nbytes(self) -> int:
+        return sum(t.numel() * t.element_size() for ts in (self.k, self.v, self.S, self.conv) for t in ts)
+
+    def reset(self, seq: Optional[int] = None):
+        sl = slice(None) if seq is None else seq
+        self.seqs[sl].zero_()
+        for t in self.S + self.conv:
+            t[sl].zero_()
+
+    def snapshot(self, seq: int = 0, with_kv: bool = False) -> MixerSnapshot:
+        n = self.length(seq)
+        return MixerSnapshot(seq, n, self.token(seq),
+                             [(k[seq, :n].clone(), v[seq, :n].clone()) for k, v in zip(self.k, self.v)] if with_kv else None,
+                             [(S[seq].clone(), c[seq].clone()) for S, c in zip(self.S, self.conv)])
+
+    def restore(self, snap: MixerSnapshot, seq: Optional[int] = None):
+        seq = snap.seq if seq is None else seq
+        self.seqs[seq, 0], self.seqs[seq, 1] = snap.length, snap.token
+        for (S, c), tS, tc in zip(snap.state, self.S, self.conv):
+            tS[seq].copy_(S)
+            tc[seq].copy_(c)
+        for (k, v), tk, tv in zip(snap.kv or [], self.k, self.v):
+            tk[seq, :snap.length].copy_(k)
+            tv[seq, :snap.length].copy_(v)
+
+    def state_dict(self, seq: int = 0) -> Dict[str, torch.Tensor]:
+        """Host-serialisable checkpoint of one sequence."""
+        s = self.snapshot(seq, with_kv=True)
+        out = {"length": torch.tensor(s.length), "token": torch.tensor(s.token)}
+        for i, ((k, v), (S, c)) in enumerate(zip(s.kv, s.state)):
+            out.update({f"k{i}": k.cpu(), f"v{i}": v.cpu(), f"S{i}": S.cpu(), f"conv{i}": c.cpu()})
+        return out
+
+    def load_state_dict(self, sd: Dict[str, torch.Tensor], seq: int = 0):
+        n = range(len(self.S))
+        self.restore(MixerSnapshot(seq, int(sd["length"]), int(sd["token"]), [(sd[f"k{i}"], sd[f"v{i}"]) for i in n],
+                                   [(sd[f"S{i}"], sd[f"conv{i}"]) for i in n]), seq)

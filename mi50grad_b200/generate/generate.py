@@ -160,25 +160,23 @@ class TextGenerator:
         self.engine.cleanup()
 
 
-def _make_engine(model_dir: str, device_ids, max_seq_len: int):
+def _make_engine(model_dir: str, device_ids, max_seq_len: int, **engine_kw):
     import torch.distributed as dist
-    from ..engine.engine import InferenceEngine
     from ..engine.tp_engine import TPInferenceEngine
-    from ..loaders import load_any
-    loader = load_any(model_dir)
-    cfg = loader.config
+    from ..models.registry import architecture_of, build_engine
     tp = dist.get_world_size() if dist.is_available() and dist.is_initialized() else 1
-    rank = dist.get_rank() if tp > 1 else 0
-    if tp > 1:
-        eng = TPInferenceEngine(cfg, device_ids, max_seq_len)
-        for i in range(cfg.num_hidden_layers):
-            eng.load_layer_weights(i, loader.load_layer(i, tp, rank), sharded=True)
-        eng.load_lm_head(loader.load_lm_head(tp, rank), sharded=True)
-    else:
-        eng = InferenceEngine(cfg, (device_ids or [0])[0], max_seq_len)
-        for i in range(cfg.num_hidden_layers):
-            eng.load_layer_weights(i, loader.load_layer(i))
-        eng.load_lm_head(loader.load_lm_head())
+    if tp == 1:
+        return build_engine(model_dir, (device_ids or [0])[0], max_seq_len, **engine_kw)
+    rank = dist.get_rank()
+    arch = architecture_of(model_dir)
+    if not arch.tensor_parallel:
+        raise NotImplementedError(f"{arch.name} runs on one GPU")
+    loader = arch.make_loader(model_dir)
+    cfg = loader.config
+    eng = TPInferenceEngine(cfg, device_ids, max_seq_len)
+    for i in range(cfg.num_hidden_layers):
+        eng.load_layer_weights(i, loader.load_layer(i, tp, rank), sharded=True)
+    eng.load_lm_head(loader.load_lm_head(tp, rank), sharded=True)
     eng.load_embedding(loader.load_embedding())
     eng.load_final_norm(loader.load_final_norm())
     return eng, loader

@@ -290,5 +290,10 @@ def load_compressed_tensors(model_dir: str, config: QwenConfig, group_size: int 
     return CompressedTensorsLoader(model_dir, config, group_size)
 
 
-def load_any(model_dir: str, config: Optional[QwenConfig] = None) -> CheckpointLoader:
+def load_any(model_dir: str, config=None):
+    """The loader of whatever architecture the directory's config.json names (a directory without one is
+    read as the hybrid decoder, with the caller's config)."""
+    if config is None or (Path(model_dir) / "config.json").exists():
+        from ..models.registry import architecture_of
+        return architecture_of(model_dir).make_loader(model_dir, config)
     return CheckpointLoader(model_dir, config)

@@ -511,3 +511,76 @@ def wait_self_test(wait_us: int = 2000) -> dict:
     torch.cuda.synchronize(dev)
     st = status.tolist()
     return {"code": st[0], "kernel": st[1], "peer": st[2], "epoch": st[3]}
+
+
+# ---------------------------------------------------------------------------
+# Dense-weight, post-norm decoder path (csrc/mixers.cuh)
+# ---------------------------------------------------------------------------
+
+def _dt(t: torch.Tensor) -> int:
+    return {torch.bfloat16: L.DT_BF16, torch.float32: L.DT_F32}[t.dtype]
+
+
+def post_norm_input(h: torch.Tensor, m: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None,
+                    ss: Optional[torch.Tensor] = None, hout: Optional[torch.Tensor] = None, eps: float = 1e-6) -> L.PostNorm:
+    """Input descriptor of `gemv_dense`: x = h + m * rsqrt(sum(ss[row]) / H + eps) * w, also stored to hout."""
+    pn = L.PostNorm()
+    pn.h, pn.m, pn.w, pn.ss, pn.hout = L.ptr(h), L.ptr(m), L.ptr(w), L.ptr(ss), L.ptr(hout)
+    pn.np, pn.H, pn.eps = (0 if ss is None else ss.shape[1]), h.shape[1], eps
+    return pn
+
+
+def gemv_dense(lin, x: Optional[torch.Tensor], out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0,
+               pn: Optional[L.PostNorm] = None, rows: Optional[int] = None, ss_out: Optional[torch.Tensor] = None):
+    """1..8 rows times a `MixerLinear`-like object (.w [N][ldw], .K, .N, .rpc); bf16 or fp32."""
+    p = L.DenseGemvParams()
+    p.w, p.ldw, p.K, p.N, p.rpc, p.dt = lin.w.data_ptr(), lin.w.stride(0), lin.K, lin.N, lin.rpc, _dt(lin.w)
+    if x is not None:
+        p.x, p.ldx, p.rows = x.data_ptr(), x.stride(0), x.shape[0]
+    else:
+        p.pn, p.rows = pn, rows
+    p.out, p.ldo, p.mode, p.softcap = out.data_ptr(), out.stride(0), mode, softcap
+    if ss_out is not None:
+        p.ss_out, p.ss_np = ss_out.data_ptr(), ss_out.shape[1]
+    L.check(L.lib().b2_gemv_dense(C.byref(p), L.stream()), "gemv_dense")
+    return out
+
+
+def gemm_f32(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0):
+    """out[t][n] = x[t] . w[n] in true fp32."""
+    p = L.GemmF32Params()
+    p.w, p.x, p.out, p.ldw, p.ldx, p.ldo = w.data_ptr(), x.data_ptr(), out.data_ptr(), w.stride(0), x.stride(0), out.stride(0)
+    p.K, p.N, p.T, p.mode, p.softcap = x.shape[1], w.shape[0], x.shape[0], mode, softcap
+    L.check(L.lib().b2_gemm_f32(C.byref(p), L.stream()), "gemm_f32")
+    return out
+
+
+def post_norm_(h: torch.Tensor, m: Optional[torch.Tensor], w: Optional[torch.Tensor], xb: torch.Tensor, eps: float,
+               final_w: Optional[torch.Tensor] = None):
+    """h += rmsnorm(m) * w in place; xb = h, or rmsnorm(h) * final_w."""
+    vp = lambda t: C.c_void_p(L.ptr(t))
+    L.check(L.lib().b2_post_norm(vp(h), vp(m), vp(w), vp(final_w), vp(xb), xb.stride(0), h.shape[0], h.shape[1], C.c_float(eps),
+                                 _dt(xb), L.stream()), "post_norm")
+    return h
+
+
+def gemm_bf16_tc(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, epi: int = L.TC_EPI_STORE_F32,
+                 t_tile: Optional[int] = None, softcap: float = 0.0):
+    """out[t][n] (epi) = x[t] . w[n] for bf16 operands on the tcgen05 tensor cores; any K (row strides
+    multiples of 8)."""
+    T, dev = x.shape[0], x.device
+    st = _tc_status.get(dev)
+    if st is None:
+        st = _tc_status[dev] = torch.zeros(64, dtype=torch.int32, device=dev)
+    p = L.GemmTcParams()
+    p.K, p.T, p.t_tile, p.epi = x.shape[1], T, t_tile or min(256, -(-T // 16) * 16), epi
+    p.n_valid = w.shape[0] // 2 if epi == L.TC_EPI_SILU_PAIR else w.shape[0]
+    p.ldo, p.out, p.status, p.bf16, p.softcap = out.stride(0), out.data_ptr(), st.data_ptr(), 1, softcap
+    L.check(L.lib().b2_gemm_f16_tc(C.byref(p), C.c_void_p(w.data_ptr()), w.stride(0), C.c_void_p(x.data_ptr()),
+                                   x.stride(0), L.stream()), "gemm_bf16_tc")
+    return out
+
+
+def mix_op(name: str, layer: L.MixLayer, run: L.MixRun):
+    """Launch one mixer kernel: 'mix_prepare', 'window_attn_decode', 'window_attn_rows', 'ssd_step', 'ssd_chunk'."""
+    L.check(getattr(L.lib(), "b2_" + name)(C.byref(layer), C.byref(run), L.stream()), name)

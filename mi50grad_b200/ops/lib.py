@@ -25,10 +25,12 @@ MAX_ROWS = 8
 EPI_STORE_F16, EPI_SILU_PAIR, EPI_STORE_F32, EPI_FINISH = 0, 1, 2, 3
 FIN_NO_COMM, FIN_NO_H_WRITE, FIN_SAVE_EXTRA, FIN_ADD_EXTRA, FIN_NO_NORM = 1, 2, 4, 8, 16
 FIN_TEST_WITHHOLD_SIGNAL = 32
-LIN_INT4, LIN_F16, LIN_NONE = 0, 1, 2
+LIN_INT4, LIN_F16, LIN_NONE, LIN_BF16, LIN_F32 = 0, 1, 2, 3, 4
+DT_BF16, DT_F32 = 0, 1
+DG_STORE, DG_SILU_PAIR, DG_STORE_F32 = 0, 1, 2
 STEP_EMBED_TOKENS, STEP_LM_HEAD, STEP_ARGMAX, STEP_ADVANCE, STEP_NO_COMMIT_DELTA = 1, 2, 4, 8, 16
 STEP_MATERIALIZE_XN = 32
-STEP_SPEC, STEP_GEMM_PATH = 64, 128
+STEP_SPEC, STEP_GEMM_PATH, STEP_HEAD_LAST = 64, 128, 256
 
 vp, i32, f32, i64 = C.c_void_p, C.c_int, C.c_float, C.c_longlong
 
@@ -117,7 +119,7 @@ class GemmTcParams(C.Structure):
                 ("gshift", i32), ("T", i32), ("t_tile", i32), ("n_valid", i32), ("ldo", i32), ("epi", i32),
                 ("stages", i32), ("out", vp), ("status", vp), ("m_halves", i32), ("dense", i32),
                 ("push", vp * MAX_TP), ("epoch", vp), ("part_stride", i64), ("push_tp", i32), ("push_rank", i32),
-                ("push_per", C.c_uint), ("k_splits", i32), ("cta_pair", i32), ("pad3", i32)]
+                ("push_per", C.c_uint), ("k_splits", i32), ("cta_pair", i32), ("bf16", i32), ("softcap", f32), ("pad3", i32)]
 
 
 TC_EPI_STORE_F16, TC_EPI_SILU_PAIR, TC_EPI_STORE_F32, TC_EPI_RESID_F32 = 0, 1, 2, 3
@@ -198,7 +200,53 @@ class ModelDesc(C.Structure):
                 ("chain_scratch", vp), ("chain_counters", vp), ("chain_act_cols", i32), ("use_chain", i32),
                 ("chain_tag_h", vp), ("chain_tag_ss", vp), ("chain_tag_act", vp),
                 ("q8_xq", vp), ("q8_sx", vp), ("q8_gate", vp), ("q8_up", vp), ("q8_down", vp), ("q8_xn", vp),
-                ("comm", CommCtx)]
+                ("comm", CommCtx), ("mixer", vp)]
+
+
+class PostNorm(C.Structure):
+    _fields_ = [("h", vp), ("m", vp), ("w", vp), ("ss", vp), ("hout", vp), ("np", i32), ("H", i32), ("eps", f32), ("pad", i32)]
+
+
+class DenseGemvParams(C.Structure):
+    _fields_ = [("w", vp), ("x", vp), ("pn", PostNorm), ("out", vp), ("ss_out", vp), ("ldw", i32), ("ldx", i32), ("K", i32),
+                ("N", i32), ("rows", i32), ("ldo", i32), ("mode", i32), ("dt", i32), ("rpc", i32), ("ss_np", i32),
+                ("softcap", f32), ("pad", i32)]
+
+
+class GemmF32Params(C.Structure):
+    _fields_ = [("w", vp), ("x", vp), ("out", vp), ("ldw", i32), ("ldx", i32), ("K", i32), ("N", i32), ("T", i32), ("ldo", i32),
+                ("mode", i32), ("pad", i32), ("softcap", f32), ("pad1", i32)]
+
+
+class MixLayer(C.Structure):
+    _fields_ = [("H", i32), ("G", i32), ("d", i32), ("dp", i32), ("rot", i32), ("window", i32),
+                ("attn_scale", f32), ("left_scale", f32), ("right_scale", f32), ("eps", f32),
+                ("q_norm", vp), ("k_norm", vp), ("cos_tab", vp), ("sin_tab", vp), ("kcache", vp), ("vcache", vp),
+                ("heads", i32), ("P", i32), ("N", i32), ("groups", i32), ("ngroups", i32), ("taps", i32),
+                ("conv_w", vp), ("conv_b", vp), ("dt_bias", vp), ("A_log", vp), ("D", vp), ("norm_w", vp),
+                ("state", vp), ("conv_state", vp),
+                ("off_q", i32), ("off_k", i32), ("off_z", i32), ("off_x", i32), ("off_dt", i32), ("max_seq", i32)]
+
+
+class MixRun(C.Structure):
+    _fields_ = [("proj", vp), ("ld_proj", i32), ("dt", i32), ("rows", vp), ("seq_rows", vp), ("n_rows", i32), ("n_seqs", i32),
+                ("qbuf", vp), ("xbc", vp), ("ld_xbc", i32), ("pad", i32), ("dtb", vp), ("ld_dt", i32), ("splits", i32),
+                ("ubuf", vp), ("ld_u", i32), ("fuse_norm", i32), ("out", vp), ("ldo", i32), ("commit", i32),
+                ("attn_scratch", vp), ("attn_counters", vp), ("ssd_counters", vp),
+                ("chunk_state", vp), ("chunk_prev", vp), ("chunk_decay", vp)]
+
+
+class MixerLayerDesc(C.Structure):
+    _fields_ = [("mix", MixLayer), ("in_proj", LinearDesc), ("out_proj", LinearDesc), ("gate_up", LinearDesc), ("down", LinearDesc),
+                ("norm1", vp), ("norm2", vp)]
+
+
+class MixerModelDesc(C.Structure):
+    _fields_ = [("layers", vp), ("final_norm", vp), ("softcap", f32), ("dt", i32), ("ss_np", i32), ("ld_x", i32),
+                ("ld_xbc", i32), ("ld_dt", i32), ("ld_u", i32), ("ld_act", i32), ("scratch_rows", i32), ("pad", i32),
+                ("m", vp), ("p_m", vp), ("qbuf", vp), ("xbc", vp), ("dtb", vp), ("ubuf", vp),
+                ("attn_scratch", vp), ("attn_counters", vp), ("ssd_counters", vp),
+                ("chunk_state", vp), ("chunk_prev", vp), ("chunk_decay", vp)]
 
 
 _SIZE_CHECKS = {
@@ -207,6 +255,8 @@ _SIZE_CHECKS = {
     "b2_sizeof_delta_params": DeltaParams, "b2_sizeof_argmax_params": ArgmaxParams,
     "b2_sizeof_linear_desc": LinearDesc, "b2_sizeof_layer_desc": LayerDesc,
     "b2_sizeof_model_desc": ModelDesc, "b2_sizeof_spec_stage": SpecStage, "b2_sizeof_sample_params": SampleParams, "b2_sizeof_quant8_params": Quant8Params, "b2_sizeof_act_quant_params": ActQuantParams, "b2_sizeof_gemm_tc_params": GemmTcParams, "b2_sizeof_row_meta": RowMeta, "b2_sizeof_seq_state": SeqState,
+    "b2_sizeof_dense_gemv_params": DenseGemvParams, "b2_sizeof_gemm_f32_params": GemmF32Params, "b2_sizeof_mix_layer": MixLayer,
+    "b2_sizeof_mix_run": MixRun, "b2_sizeof_mixer_layer_desc": MixerLayerDesc, "b2_sizeof_mixer_model_desc": MixerModelDesc,
     "b2_sizeof_chain_params": ChainParams, "b2_sizeof_chain_op": ChainOp,
 }
 
@@ -241,6 +291,8 @@ def lib() -> C.CDLL:
     _lib.b2_driver_total_exchanges.restype = i64
     _lib.b2_chain_scratch_floats.restype = i64
     _lib.b2_gemv_int4_smem.restype = C.c_size_t
+    for fn in ("b2_window_attn_scratch", "b2_ssd_chunk_state_floats", "b2_ssd_chunk_prev_bytes"):
+        getattr(_lib, fn).restype = i64
     return _lib
 
 
