@@ -321,8 +321,10 @@ def main():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-like-for-like", action="store_true",
                     help="skip the second timed run with fp16 attention weights (the published numbers' checkpoint layout)")
-    ap.add_argument("--mode", default="decode", choices=["decode", "batch-spec"],
-                    help="batch-spec: batched decode with per-step draft verification (batch x ctx, --draft tokens)")
+    ap.add_argument("--mode", default="decode", choices=["decode", "batch-spec", "degedra"],
+                    help="batch-spec: batched decode with per-step draft verification (batch x ctx, --draft tokens); "
+                         "degedra: the Degedra decoder at a few layer sizes beside the hybrid decoder of equal size")
+    ap.add_argument("--sizes", default="2k,4k,5k", help="degedra: layer sizes, with commas between them")
     ap.add_argument("--batch", type=int, default=16)
     ap.add_argument("--ctx", type=int, default=4096)
     ap.add_argument("--draft", type=int, default=4)
@@ -352,6 +354,12 @@ def main():
     if args.impl == "torch":
         return torch_baseline(args, cfg, world, rank, local)
     from mi50grad_b200.engine.tp_engine import TPInferenceEngine
+    if args.mode == "degedra":
+        if world != 1:
+            raise SystemExit("--mode degedra runs on one GPU")
+        from mi50grad_b200.bench.degedra import run
+        print(json.dumps(run(args.steps, args.warmup, args.sizes.split(","), ClockSampler(local))))
+        return 0
     if args.mode == "batch-spec":
         return batch_spec(args, cfg, world, rank, local)
     max_seq = max(1024, args.prompt_len + args.steps + args.warmup + 640)

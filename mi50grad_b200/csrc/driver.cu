@@ -399,7 +399,7 @@ static int argmax_advance(Driver* d, bool many, int rows, int n_seqs, int flags,
         d->launches++;
     }
     if (flags & STEP_ADVANCE) {
-        CK(b2_advance(m.seqs, nullptr, n_seqs, 1, s));
+        CK(b2_advance(m.seqs, many ? m.p_rows : m.rows, m.seq_rows, n_seqs, s));
         d->launches++;
     }
     return 0;

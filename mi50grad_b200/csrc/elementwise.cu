@@ -39,14 +39,15 @@ B2_API int b2_prepare_rows(const void* tmpl, const void* seqs, void* rows, int n
     return cudaGetLastError();
 }
 
-// advance: len += add[seq] for every sequence (after a step has been committed)
-__global__ void advance_kernel(SeqState* seqs, const int* __restrict__ add, int n, int add_const) {
+// advance: len += 1 of every sequence that had rows in the step (after the step has been committed); launched
+// sequence i is the one rows[seq_rows[i]] belongs to
+__global__ void advance_kernel(SeqState* seqs, const RowMeta* __restrict__ rows, const int* __restrict__ seq_rows, int n) {
     pdl_launch_dependents();
     int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) seqs[i].len += add ? add[i] : add_const;
+    if (i < n) seqs[rows[seq_rows[i]].seq].len += 1;
 }
-B2_API int b2_advance(void* seqs, const int* add, int n, int add_const, cudaStream_t s) {
-    advance_kernel<<<(n + 63) / 64, 64, 0, s>>>((SeqState*)seqs, add, n, add_const);
+B2_API int b2_advance(void* seqs, const void* rows, const int* seq_rows, int n, cudaStream_t s) {
+    advance_kernel<<<(n + 63) / 64, 64, 0, s>>>((SeqState*)seqs, (const RowMeta*)rows, seq_rows, n);
     return cudaGetLastError();
 }
 

@@ -43,6 +43,7 @@ def lazy_norm(h: torch.Tensor, ss: torch.Tensor, w: torch.Tensor, eps: float = 1
     ln = L.LazyNorm()
     ln.h, ln.ss, ln.w = h.data_ptr(), ss.data_ptr(), w.data_ptr()
     ln.np, ln.H, ln.eps = ss.shape[1], h.shape[1], eps
+    ln.tensors = (h, ss, w)      # the descriptor holds addresses only: keep the memory until it is dropped
     return ln
 
 
@@ -527,6 +528,7 @@ def post_norm_input(h: torch.Tensor, m: Optional[torch.Tensor] = None, w: Option
     pn = L.PostNorm()
     pn.h, pn.m, pn.w, pn.ss, pn.hout = L.ptr(h), L.ptr(m), L.ptr(w), L.ptr(ss), L.ptr(hout)
     pn.np, pn.H, pn.eps = (0 if ss is None else ss.shape[1]), h.shape[1], eps
+    pn.tensors = (h, m, w, ss, hout)
     return pn
 
 

@@ -105,6 +105,17 @@ def test_two_sequences_with_independent_lengths(setup):
     assert eng.states.lengths() == [16, 9]
 
 
+def test_decoding_a_slot_other_than_the_first(setup):
+    """The step advances the sequences it decodes, whichever slots they are in."""
+    cfg, mw, eng, orc = setup
+    eng.states.reset(); orc.reset()
+    p = _prompt(cfg, 9, seed=11)
+    t = eng.prefill_tokens(p, seq=1)
+    out = eng.decode_tokens(6, seqs=[1], graph=True).cpu()
+    ref, _ = orc.greedy_generate(p, 7, seq=1)
+    assert [t] + out[:, 0].tolist() == ref and eng.states.lengths() == [0, 15]
+
+
 def test_snapshot_restore_rolls_back_deltanet(setup):
     cfg, mw, eng, orc = setup
     ids = _prompt(cfg, 10, seed=7)
