@@ -13,74 +13,157 @@
 #include "mixers.cuh"
 
 // ---------------------------------------------------------------------------
-// prepare: grid (2 + convolution blocks, rows)
+// prepare: one-dimensional grid.  First (q_slices + 1) CTAs per row: slices of the query heads, then the keys;
+// every one of them sums the squares of its whole projection.  Then the convolution: column blocks of 512
+// channels times tiles of conv_rows rows.
 // ---------------------------------------------------------------------------
 #define MP_THREADS 256
-#define MP_CONV 4                // channels per thread
+#define MP_COLS (2 * MP_THREADS)
+#define MP_MAX_ROWS 8            // rows of a convolution tile
+#define MP_TAPS 4                // taps whose weights stay in registers
 
 template <typename T>
-__global__ void __launch_bounds__(MP_THREADS) mix_prepare_kernel(const MixLayer L, const MixRun R) {
-    extern __shared__ float mp_v[];              // the projection part of one row
+__device__ __forceinline__ void mp_heads(const MixLayer& L, const MixRun& R, int r, int slice, int q_slices, float* sv, float* red) {
+    const int tid = threadIdx.x;
+    const bool is_q = slice < q_slices;
+    const RowMeta rm = R.rows[r];
+    const int heads = is_q ? L.H : L.G, n = heads * L.d, off = is_q ? L.off_q : L.off_k;
+    const int per = is_q ? (heads + q_slices - 1) / q_slices : heads;
+    const int h0 = is_q ? slice * per : 0, h1 = min(heads, h0 + per), i0 = h0 * L.d, i1 = h1 * L.d;
+    const T* src = (const T*)R.proj + (size_t)r * R.ld_proj + off;
+    const float* nw = is_q ? L.q_norm : L.k_norm;
+    const size_t slot = ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
+    T* dst = is_q ? (T*)R.qbuf + (size_t)r * L.H * L.dp : (T*)L.kcache + slot;
+    T* vdst = (T*)L.vcache + slot;
+    constexpr int V = 16 / sizeof(T);
+    const bool vec = ((off | R.ld_proj | n) & (V - 1)) == 0;
+    pdl_wait();
+    float ss = 0.f;
+    if (vec) {
+#pragma unroll 2
+        for (int i = tid * V; i < n; i += MP_THREADS * V) {
+            const uint4 u = *(const uint4*)(src + i);
+            const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                const float v = sizeof(T) == 4 ? __uint_as_float(w[e & 3])
+                                               : __uint_as_float((e & 1) ? (w[(e >> 1) & 3] & 0xffff0000u) : (w[(e >> 1) & 3] << 16));
+                ss += v * v;
+                if (i + e >= i0 && i + e < i1) sv[i + e - i0] = v;
+            }
+        }
+    } else
+        for (int i = tid; i < n; i += MP_THREADS) {
+            const float v = ld_f(src + i);
+            ss += v * v;
+            if (i >= i0 && i < i1) sv[i - i0] = v;
+        }
+    const float inv = rsqrtf(block_sum(ss, red) / (float)n + L.eps);      // (its barriers also publish sv)
+    const int half = L.rot >> 1;
+    const float* ct = L.cos_tab + (size_t)rm.pos * half;
+    const float* st = L.sin_tab + (size_t)rm.pos * half;
+#pragma unroll 2
+    for (int i = tid; i < (h1 - h0) * L.dp; i += MP_THREADS) {
+        const int hd = i / L.dp, e = i - hd * L.dp, j = hd * L.d + e;
+        float o = 0.f, raw = 0.f;
+        if (e < L.d) {
+            raw = sv[j];
+            o = raw * inv * nw[i0 + j];
+            if (e < L.rot) {
+                const bool first = e < half;
+                const int a = first ? e : e - half, jo = first ? j + half : j - half;
+                const float other = sv[jo] * inv * nw[i0 + jo];
+                o = first ? o * ct[a] - other * st[a] : o * ct[a] + other * st[a];
+            }
+        }
+        dst[h0 * L.dp + i] = to_t<T>(o);
+        if (!is_q) vdst[i] = to_t<T>(raw);
+    }
+}
+
+// two adjacent elements (one 2 x sizeof(T) load when `pair`: the address is aligned to it)
+template <typename T>
+__device__ __forceinline__ float2 mp_ld2(const T* p, bool pair, bool second) {
+    if (pair) {
+        if constexpr (sizeof(T) == 4) return *(const float2*)p;
+        else return __bfloat1622float2(*(const __nv_bfloat162*)p);
+    }
+    return make_float2(ld_f(p), second ? ld_f(p + 1) : 0.f);
+}
+
+template <typename T>
+__device__ __forceinline__ void mp_conv(const MixLayer& L, const MixRun& R, int blk, int r0, int rows) {
+    __shared__ int s_local[MP_MAX_ROWS], s_seq[MP_MAX_ROWS];
+    const int tid = threadIdx.x, C = L.heads * L.P + 2 * L.groups * L.N, c = blk * MP_COLS + 2 * tid, K = L.taps - 1;
+    if (tid < rows) {
+        // rows of the same sequence in front of this one in the launch, as far as the taps reach
+        const int r = r0 + tid, seq = R.rows[r].seq;
+        int local = 0;
+        while (local < K && r - local - 1 >= 0 && R.rows[r - local - 1].seq == seq) ++local;
+        s_local[tid] = local; s_seq[tid] = seq;
+    }
+    const bool in = c < C, second = c + 1 < C;
+    const bool pair = second && ((L.off_x | R.ld_proj | C) & 1) == 0, pair_out = second && (R.ld_xbc & 1) == 0;
+    float b0 = 0.f, b1 = 0.f, w0[MP_TAPS], w1[MP_TAPS];
+    const bool regs = L.taps <= MP_TAPS;
+    if (in) {
+        b0 = L.conv_b[c]; b1 = second ? L.conv_b[c + 1] : 0.f;
+#pragma unroll
+        for (int j = 0; j < MP_TAPS; ++j) {
+            w0[j] = (regs && j < L.taps) ? L.conv_w[(size_t)c * L.taps + j] : 0.f;
+            w1[j] = (regs && j < L.taps && second) ? L.conv_w[(size_t)(c + 1) * L.taps + j] : 0.f;
+        }
+    }
+    pdl_wait();
+    __syncthreads();
+    if (blk == 0)
+        for (int i = tid; i < rows * L.heads; i += MP_THREADS) {
+            const int r = r0 + i / L.heads, h = i % L.heads;
+            R.dtb[(size_t)r * R.ld_dt + h] = softplus_p(ld_f((const T*)R.proj + (size_t)r * R.ld_proj + L.off_dt + h) + L.dt_bias[h]);
+        }
+    if (!in) return;
+    for (int i = 0; i < rows; ++i) {
+        const int r = r0 + i, local = s_local[i];
+        const T* row = (const T*)R.proj + (size_t)r * R.ld_proj + L.off_x + c;
+        const T* hist = (const T*)L.conv_state + (size_t)s_seq[i] * K * C + c;
+        auto tap = [&](int j) {                              // weight j belongs to the input K - j tokens back
+            const int back = K - j;
+            return back <= local ? mp_ld2(row - (size_t)back * R.ld_proj, pair, second)
+                                 : mp_ld2(hist + (size_t)(K - (back - local)) * C, pair, second);
+        };
+        float a0 = b0, a1 = b1;
+        if (regs) {
+            float2 v[MP_TAPS];
+#pragma unroll
+            for (int j = 0; j < MP_TAPS; ++j) v[j] = j < L.taps ? tap(j) : make_float2(0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j < MP_TAPS; ++j) { a0 = fmaf(w0[j], v[j].x, a0); a1 = fmaf(w1[j], v[j].y, a1); }
+        } else
+            for (int j = 0; j < L.taps; ++j) {
+                const float2 v = tap(j);
+                a0 = fmaf(L.conv_w[(size_t)c * L.taps + j], v.x, a0);
+                if (second) a1 = fmaf(L.conv_w[(size_t)(c + 1) * L.taps + j], v.y, a1);
+            }
+        T* out = (T*)R.xbc + (size_t)r * R.ld_xbc + c;
+        const T o0 = to_t<T>(silu_p(a0)), o1 = to_t<T>(silu_p(a1));
+        if (pair_out) {
+            if constexpr (sizeof(T) == 4) *(float2*)out = make_float2(o0, o1);
+            else { __nv_bfloat162 h; h.x = o0; h.y = o1; *(__nv_bfloat162*)out = h; }
+        } else { out[0] = o0; if (second) out[1] = o1; }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(MP_THREADS) mix_prepare_kernel(const MixLayer L, const MixRun R, int q_slices, int col_blocks, int conv_rows) {
+    extern __shared__ float mp_v[];              // the heads a CTA rotates
     __shared__ float red[32];
     pdl_launch_dependents();
-    const int r = blockIdx.y, part = blockIdx.x, tid = threadIdx.x;
-    const RowMeta rm = R.rows[r];
-    const T* row = (const T*)R.proj + (size_t)r * R.ld_proj;
-    if (part < 2) {
-        // ---- queries (part 0) or keys and values (part 1)
-        const int heads = part == 0 ? L.H : L.G, n = heads * L.d;
-        const T* src = row + (part == 0 ? L.off_q : L.off_k);
-        const float* nw = part == 0 ? L.q_norm : L.k_norm;
-        T* dst = part == 0 ? (T*)R.qbuf + (size_t)r * L.H * L.dp
-                           : (T*)L.kcache + ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
-        T* vdst = (T*)L.vcache + ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
-        pdl_wait();
-        float ss = 0.f;
-        for (int i = tid; i < n; i += MP_THREADS) { const float v = ld_f(src + i); mp_v[i] = v; ss += v * v; }
-        const float inv = rsqrtf(block_sum(ss, red) / (float)n + L.eps);      // (its barriers also publish mp_v)
-        const int half = L.rot >> 1;
-        const float* ct = L.cos_tab + (size_t)rm.pos * half;
-        const float* st = L.sin_tab + (size_t)rm.pos * half;
-        for (int i = tid; i < heads * L.dp; i += MP_THREADS) {
-            const int hd = i / L.dp, e = i % L.dp, j = hd * L.d + e;
-            float o = 0.f, raw = 0.f;
-            if (e < L.d) {
-                raw = mp_v[j];
-                o = raw * inv * nw[j];
-                if (e < L.rot) {
-                    const bool first = e < half;
-                    const int a = first ? e : e - half, jo = first ? j + half : j - half;
-                    const float other = mp_v[jo] * inv * nw[jo];
-                    o = first ? o * ct[a] - other * st[a] : o * ct[a] + other * st[a];
-                }
-            }
-            dst[i] = to_t<T>(o);
-            if (part == 1) vdst[i] = to_t<T>(raw);
-        }
-        return;
-    }
-    // ---- convolution over time of x | B | C, and (first block) the step sizes
-    const int C = L.heads * L.P + 2 * L.groups * L.N;
-    const T* hist = (const T*)L.conv_state + (size_t)rm.seq * (L.taps - 1) * C;
-    // rows of this sequence in front of r in this launch, as far as the taps reach
-    int local = 0;
-    while (local < L.taps - 1 && r - local - 1 >= 0 && R.rows[r - local - 1].seq == rm.seq) ++local;
-    pdl_wait();
-    if (part == 2 && tid < L.heads)
-        for (int h = tid; h < L.heads; h += MP_THREADS)
-            R.dtb[(size_t)r * R.ld_dt + h] = softplus_p(ld_f(row + L.off_dt + h) + L.dt_bias[h]);
-#pragma unroll
-    for (int u = 0; u < MP_CONV; ++u) {
-        const int c = ((part - 2) * MP_CONV + u) * MP_THREADS + tid;
-        if (c >= C) continue;
-        float a = L.conv_b[c];
-        for (int j = L.taps - 1; j >= 0; --j) {                 // j tokens back; oldest first
-            const float v = j <= local ? ld_f(row - (size_t)j * R.ld_proj + L.off_x + c)
-                                       : ld_f(hist + (size_t)(L.taps - 1 - (j - local)) * C + c);
-            a = fmaf(L.conv_w[(size_t)c * L.taps + (L.taps - 1 - j)], v, a);
-        }
-        ((T*)R.xbc)[(size_t)r * R.ld_xbc + c] = to_t<T>(silu_p(a));
-    }
+    const int nh = R.n_rows * (q_slices + 1);
+    int b = blockIdx.x;
+    if (b < nh) { mp_heads<T>(L, R, b / (q_slices + 1), b % (q_slices + 1), q_slices, mp_v, red); return; }
+    b -= nh;
+    const int r0 = (b / col_blocks) * conv_rows;
+    mp_conv<T>(L, R, b % col_blocks, r0, min(conv_rows, R.n_rows - r0));
 }
 
 B2_API int b2_mix_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s) {
@@ -88,15 +171,21 @@ B2_API int b2_mix_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s) {
         l->taps < 1 || l->groups < 1 || l->heads % l->groups)
         return cudaErrorInvalidValue;
     const int C = l->heads * l->P + 2 * l->groups * l->N;
-    dim3 grid(2 + (C + MP_THREADS * MP_CONV - 1) / (MP_THREADS * MP_CONV), r->n_rows);
-    const size_t smem = (size_t)(l->H > l->G ? l->H : l->G) * l->d * sizeof(float);
+    // few rows: cut the query heads so that a slice is one pass of a CTA; many rows fill the GPU as they are
+    int qs = r->n_rows <= B2_MAX_ROWS ? (l->H * l->d + 511) / 512 : 1;
+    if (qs > l->H) qs = l->H;
+    const int per = (l->H + qs - 1) / qs;
+    qs = (l->H + per - 1) / per;
+    const int cb = (C + MP_COLS - 1) / MP_COLS, cr = r->n_rows <= B2_MAX_ROWS ? 1 : MP_MAX_ROWS;
+    const dim3 grid(r->n_rows * (qs + 1) + cb * ((r->n_rows + cr - 1) / cr));
+    const size_t smem = (size_t)(per > l->G ? per : l->G) * l->d * sizeof(float);
     static SmemOptIn opt[2];
     if (r->dt == DT_BF16) {
         if (int e = opt[0].ensure((const void*)mix_prepare_kernel<bf16>, smem)) return e;
-        return launch_pdl(mix_prepare_kernel<bf16>, grid, dim3(MP_THREADS), smem, s, *l, *r);
+        return launch_pdl(mix_prepare_kernel<bf16>, grid, dim3(MP_THREADS), smem, s, *l, *r, qs, cb, cr);
     }
     if (int e = opt[1].ensure((const void*)mix_prepare_kernel<float>, smem)) return e;
-    return launch_pdl(mix_prepare_kernel<float>, grid, dim3(MP_THREADS), smem, s, *l, *r);
+    return launch_pdl(mix_prepare_kernel<float>, grid, dim3(MP_THREADS), smem, s, *l, *r, qs, cb, cr);
 }
 
 // ---------------------------------------------------------------------------

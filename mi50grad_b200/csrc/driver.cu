@@ -33,8 +33,8 @@ struct LinearDesc {
     int kind;
     int K, N;                     // logical in/out features (N: valid outputs)
     int KB, NTL, G, off32, gshift;
-    int k_splits, L;              // int4 launch shape
-    int ldw, kslice;              // f16 launch shape
+    int k_splits, L;              // int4 launch shape; bf16 / fp32: L = outputs per CTA of a launch with more than two rows
+    int ldw, kslice;              // f16 launch shape; bf16 / fp32: kslice = outputs per CTA with one or two rows
     int pad;
     const void* w;                // qfrag or fp16 weights
     const void* sz;               // szfrag
@@ -129,8 +129,8 @@ struct MixerModelDesc {
     const float* final_norm;
     float softcap; int dt;
     int ss_np, ld_x;              // partial sums per row; row stride of p_xn
-    int ld_xbc, ld_dt, ld_u, ld_act, scratch_rows, pad;    // scratch_rows: rows the split-attention scratch holds
-    float* m; float* p_m;         // raw sublayer outputs [rows][H]
+    int ld_xbc, ld_dt, ld_u, ld_act, scratch_rows, m_planes;    // scratch_rows: rows the split-attention scratch holds
+    float* m; float* p_m;         // raw sublayer outputs [rows][H]; p_m: m_planes of them, max_prefill rows apart
     void* qbuf; void* xbc; float* dtb; float* ubuf;            // sized for max(max_rows, max_prefill) rows
     float* attn_scratch; int* attn_counters; int* ssd_counters;
     float* chunk_state; void* chunk_prev; float* chunk_decay;  // chunked scan (null: token by token only)
@@ -172,6 +172,7 @@ struct Driver {
     int pf_blocks = 0;                    // k-blocks per warp of the next projection that a GEMV prefetches into L2 (0: off)
     int gemv_seq = 0;                     // split-K GEMVs issued so far in the step being issued (their tags)
     int push_rows_per = 0;                // > 0 while a GEMM is issued whose pushed slices are whole token rows
+    int mixer_lazy_rows = 1;              // mixer models: up to this many rows the residual updates ride in the projections
     bool sp_now = false;                  // the many-row step being issued keeps the residual stream sequence-parallel
 };
 
@@ -738,21 +739,25 @@ static int rows_impl(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
 // ---------------------------------------------------------------------------
 // Post-norm decoders of parallel mixers.
 // ---------------------------------------------------------------------------
+static inline int mixer_rpc(const LinearDesc& L, int rows) { return rows <= DG_FMA_ROWS ? L.kslice : L.L; }
 // Decode projection; pn: the residual update its input still owes (x null), ss_out: partial sums for the next one.
 static int mixer_gemv(Driver* d, const LinearDesc& L, const void* x, int ldx, const PostNorm& pn, int rows, void* out, int ldo,
                       int mode, float* ss_out, float softcap, cudaStream_t s) {
     DenseGemvParams p;
     memset(&p, 0, sizeof(p));
     p.w = L.w; p.x = x; p.pn = pn; p.out = out; p.ss_out = ss_out; p.ldw = L.ldw; p.ldx = ldx; p.K = L.K; p.N = L.N;
-    p.rows = rows; p.ldo = ldo; p.mode = mode; p.dt = d->mx.dt; p.rpc = L.L; p.ss_np = d->mx.ss_np; p.softcap = softcap;
+    p.rows = rows; p.ldo = ldo; p.mode = mode; p.dt = d->mx.dt; p.rpc = mixer_rpc(L, rows); p.ss_np = d->mx.ss_np; p.softcap = softcap;
     d->launches++;
     return b2_gemv_dense(&p, s);
 }
 
-// Many-row projection: tcgen05 GEMM (bf16) or the fp32 GEMM.
+// Many-row projection: tcgen05 GEMM (bf16) or the fp32 GEMM.  planes (optional, in: the most planes `out` has
+// room for, max_prefill rows apart; out: the planes written): the product may be split over K.
 static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, int T, void* out, int ldo, int mode, float softcap,
-                      cudaStream_t s) {
+                      cudaStream_t s, int* planes = nullptr) {
     d->launches++;
+    const int max_ks = planes ? *planes : 1;
+    if (planes) *planes = 1;
     if (d->mx.dt == DT_F32) {
         GemmF32Params p;
         memset(&p, 0, sizeof(p));
@@ -762,14 +767,31 @@ static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, in
     }
     GemmTcParams p;
     memset(&p, 0, sizeof(p));
-    const int ctas_n = (L.N + 127) / 128;
-    int tt = T >= 256 ? 256 : ((T + 15) & ~15);
-    if (ctas_n < 148) {                                    // few output tiles: cut the tokens until the grid fills one wave
-        int need = ((T + 148 / ctas_n - 1) / (148 / ctas_n) + 15) & ~15;
-        if (need < 64) need = 64;
-        if (need < tt) tt = need;
-    }
-    p.K = L.K; p.T = T; p.t_tile = tt; p.ldo = ldo; p.out = out; p.status = d->m.tc_status; p.bf16 = 1; p.softcap = softcap;
+    // Token tile, CTA pairs and K splits: an SM takes in about 65 GB/s of operand tiles (measured, whatever the
+    // tile), so a 64-k block of a 128-output CTA costs the time of its 16 KB of weights and 128 bytes per token
+    // row it loads (half of the rows in a pair), but not less than its tensor time.
+    const int ctas_n = (L.N + 127) / 128, KB = (L.K + 63) / 64;
+    int best_t = 64, best_pair = 0, best_ks = 1;
+    double best = 1e30;
+    const int tiles[] = {64, 96, 128, 160, 192, 224, 256, 512};
+    for (int i = 0; i < 8; ++i)
+        for (int pair = 0; pair < 2; ++pair) {
+            const int t = tiles[i];
+            if (pair ? t < 256 : (t > 256 || t >= T + 64)) continue;
+            if (pair && t == 512 && T <= 256) continue;
+            const int nn = pair ? ctas_n + (ctas_n & 1) : ctas_n, nt = (T + t - 1) / t;
+            const double load = (16384.0 + (pair ? 64.0 : 128.0) * t) / 65000.0, math = t / 256.0 * 0.45;
+            const double blk = load > math ? load : math;
+            for (int ks = 1; ks <= max_ks; ++ks) {
+                const int k1 = b2_gemm_tc_splits(L.K, ks), waves = (nn * nt * k1 + 147) / 148;
+                const double cost = waves * ((KB + k1 - 1) / k1 * blk + 3.0) + (k1 > 1 ? 0.7 * k1 : 0.0);
+                if (cost < best) { best = cost; best_t = t; best_pair = pair; best_ks = ks; }
+            }
+        }
+    p.K = L.K; p.T = T; p.t_tile = best_t; p.cta_pair = best_pair; p.k_splits = best_ks;
+    if (!best_pair && p.t_tile > ((T + 15) & ~15)) p.t_tile = (T + 15) & ~15;
+    p.ldo = ldo; p.out = out; p.status = d->m.tc_status; p.bf16 = 1; p.softcap = softcap;
+    if (planes) { *planes = b2_gemm_tc_splits(L.K, best_ks); p.plane_stride = (long long)d->m.max_prefill * ldo; }
     p.n_valid = mode == DG_SILU_PAIR ? L.N / 2 : L.N;
     p.epi = mode == DG_SILU_PAIR ? TC_EPI_SILU_PAIR : (mode == DG_STORE ? TC_EPI_STORE_F16 : TC_EPI_STORE_F32);
     return b2_gemm_f16_tc(&p, L.w, L.ldw, x, ldx, s);
@@ -797,8 +819,9 @@ struct LayerCount {
     ~LayerCount() { d->layer_launches[li] = (int)(d->launches - l0); }
 };
 
-// <= 8 rows.  The residual update of a sublayer is formed by the projection that follows it, so the stream
-// alternates between two buffers; the first is chosen so that it ends in m.h.
+// <= 8 rows.  With few rows (mixer_lazy_rows) the residual update of a sublayer is formed by the projection
+// that follows it, so the stream alternates between two buffers; the first is chosen so that it ends in m.h.
+// With more rows every CTA's own copy of that work costs more than a launch that does it once.
 static int mixer_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
     const ModelDesc& m = d->m;
     const MixerModelDesc& x = d->mx;
@@ -806,48 +829,54 @@ static int mixer_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s
     if (flags & STEP_SPEC) return cudaErrorNotSupported;
     d->launches = 0; d->chain_launches = 0; d->exchanges = 0; d->pend.n = 0;
     CK(b2_prepare_rows(m.rows_tmpl, m.seqs, m.rows, rows, nullptr, s)); d->launches++;
+    const bool lazy = rows <= d->mixer_lazy_rows;
     int flips = 0;
-    for (int li = 0; li < m.n_layers; ++li) flips += (li > 0) + (d->mlayers[li].down.kind != LIN_NONE);
+    for (int li = 0; lazy && li < m.n_layers; ++li) flips += (li > 0) + (d->mlayers[li].down.kind != LIN_NONE);
     float* h = (flips & 1) ? m.h_tmp : m.h;
     float* h2 = (flips & 1) ? m.h : m.h_tmp;
     if (flags & STEP_EMBED_TOKENS) {
-        CK(b2_embed_rows(m.embed, m.row_tokens, m.rows, m.seqs, h, nullptr, 0, rows, m.H, m.vocab, x.dt, s)); d->launches++;
+        CK(b2_embed_rows(m.embed, m.row_tokens, m.rows, m.seqs, h, lazy ? nullptr : m.xn, x.ld_x, rows, m.H, m.vocab, x.dt, s));
+        d->launches++;
     } else {
         // (an ordinary stream operation in any case: the kernels below read the row table ahead of their
         // dependency wait, which is safe only if prepare_rows has completed before the first of them starts)
         if (cudaError_t e = cudaMemcpyAsync(m.h_tmp, m.h, (size_t)rows * m.H * sizeof(float), cudaMemcpyDeviceToDevice, s)) return e;
+        if (!lazy) { CK(b2_post_norm(h, nullptr, nullptr, nullptr, m.xn, x.ld_x, rows, m.H, m.eps, x.dt, 1, 0, s)); d->launches++; }
     }
     const float* owed = nullptr;                 // weights of the norm whose residual update is still owed
     int owed_np = 0;
     PostNorm none;
     memset(&none, 0, sizeof(none));
-    auto input = [&]() {
-        PostNorm pn;
-        memset(&pn, 0, sizeof(pn));
+    // a projection of the residual stream, with the owed update
+    auto project = [&](const LinearDesc& L, void* out, int ldo, int mode) -> int {
+        if (!lazy) {
+            if (owed) { CK(b2_post_norm(h, x.m, owed, nullptr, m.xn, x.ld_x, rows, m.H, m.eps, x.dt, 1, 0, s)); d->launches++; owed = nullptr; }
+            return mixer_gemv(d, L, m.xn, x.ld_x, none, rows, out, ldo, mode, nullptr, 0.f, s);
+        }
+        PostNorm pn = none;
         pn.h = h; pn.H = m.H; pn.eps = m.eps;
         if (owed) { pn.m = x.m; pn.w = owed; pn.ss = m.ss; pn.np = owed_np; pn.hout = h2; }
-        return pn;
+        CK(mixer_gemv(d, L, nullptr, 0, pn, rows, out, ldo, mode, nullptr, 0.f, s));
+        if (owed) { float* t = h; h = h2; h2 = t; owed = nullptr; }
+        return 0;
     };
-    auto settled = [&]() { if (owed) { float* t = h; h = h2; h2 = t; } owed = nullptr; };
     const MixRun r = mixer_run(d, false, rows, n_seqs, flags);
     for (int li = 0; li < m.n_layers; ++li) {
         const MixerLayerDesc& L = d->mlayers[li];
         LayerCount count(d, li);
-        CK(mixer_gemv(d, L.in_proj, nullptr, 0, input(), rows, m.proj, m.ld_proj, DG_STORE, nullptr, 0.f, s));
-        settled();
+        CK(project(L.in_proj, m.proj, m.ld_proj, DG_STORE));
         CK(b2_mix_prepare(&L.mix, &r, s)); d->launches++;
         CK(b2_window_attn_decode(&L.mix, &r, s)); d->launches++;
         CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2;
         CK(mixer_gemv(d, L.out_proj, m.attn_out, m.ld_attn, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
-        owed = L.norm1; owed_np = (m.H + L.out_proj.L - 1) / L.out_proj.L;
+        owed = L.norm1; owed_np = (m.H + mixer_rpc(L.out_proj, rows) - 1) / mixer_rpc(L.out_proj, rows);
         if (L.down.kind == LIN_NONE) continue;
-        CK(mixer_gemv(d, L.gate_up, nullptr, 0, input(), rows, m.act, x.ld_act, DG_SILU_PAIR, nullptr, 0.f, s));
-        settled();
+        CK(project(L.gate_up, m.act, x.ld_act, DG_SILU_PAIR));
         CK(mixer_gemv(d, L.down, m.act, x.ld_act, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
-        owed = L.norm2; owed_np = (m.H + L.down.L - 1) / L.down.L;
+        owed = L.norm2; owed_np = (m.H + mixer_rpc(L.down, rows) - 1) / mixer_rpc(L.down, rows);
     }
     // the last residual update and the final norm (xn feeds the head and the hidden-out interface)
-    CK(b2_post_norm(h, owed ? x.m : nullptr, owed, x.final_norm, m.xn, x.ld_x, rows, m.H, m.eps, x.dt, s)); d->launches++;
+    CK(b2_post_norm(h, owed ? x.m : nullptr, owed, x.final_norm, m.xn, x.ld_x, rows, m.H, m.eps, x.dt, 1, 0, s)); d->launches++;
     if (flags & STEP_LM_HEAD)
         CK(mixer_gemv(d, m.lm_head, m.xn, x.ld_x, none, rows, m.logits, m.ld_logits, DG_STORE_F32, nullptr, x.softcap, s));
     return argmax_advance(d, false, rows, n_seqs, flags, s);
@@ -863,7 +892,7 @@ static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
     if (flags & STEP_EMBED_TOKENS)
         CK(b2_embed_rows(m.embed, m.p_row_tokens, m.p_rows, m.seqs, m.p_h, m.p_xn, x.ld_x, T, m.H, m.vocab, x.dt, s));
     else
-        CK(b2_post_norm(m.p_h, nullptr, nullptr, nullptr, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s));
+        CK(b2_post_norm(m.p_h, nullptr, nullptr, nullptr, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, 1, 0, s));
     d->launches++;
     const MixRun r = mixer_run(d, true, T, n_seqs, flags);
     const bool one = n_seqs == 1 && x.dt == DT_BF16;
@@ -877,13 +906,15 @@ static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
         d->launches += 2;
         if (one && T >= 32 && x.chunk_state) { CK(b2_ssd_chunk(&L.mix, &r, s)); d->launches += 4; }
         else { CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2; }
-        CK(mixer_gemm(d, L.out_proj, m.p_attn, m.ld_attn, T, x.p_m, m.H, DG_STORE_F32, 0.f, s));
+        int planes = x.m_planes;
+        CK(mixer_gemm(d, L.out_proj, m.p_attn, m.ld_attn, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
         const bool ff = L.down.kind != LIN_NONE;
-        CK(b2_post_norm(m.p_h, x.p_m, L.norm1, ff ? nullptr : after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s)); d->launches++;
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm1, ff ? nullptr : after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
         if (!ff) continue;
         CK(mixer_gemm(d, L.gate_up, m.p_xn, x.ld_x, T, m.p_act, x.ld_act, DG_SILU_PAIR, 0.f, s));
-        CK(mixer_gemm(d, L.down, m.p_act, x.ld_act, T, x.p_m, m.H, DG_STORE_F32, 0.f, s));
-        CK(b2_post_norm(m.p_h, x.p_m, L.norm2, after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, s)); d->launches++;
+        planes = x.m_planes;
+        CK(mixer_gemm(d, L.down, m.p_act, x.ld_act, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm2, after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
     }
     if (flags & STEP_HEAD_LAST) {
         if (n_seqs != 1 || (flags & STEP_ADVANCE)) return cudaErrorInvalidValue;
@@ -938,6 +969,8 @@ B2_API void* b2_driver_create(const ModelDesc* m, const LayerDesc* layers) {
     // state is a small part of its 10 us.
     const char* pfs = getenv("B200GRAD_PREFETCH_STATE");
     d->pf_state = pfs && atoi(pfs) != 0;
+    const char* mlr = getenv("B200GRAD_LAZY_ROWS");
+    if (mlr) d->mixer_lazy_rows = atoi(mlr);
     const char* pf = getenv("B200GRAD_L2_PREFETCH");
     d->pf_blocks = pf ? atoi(pf) : 0;
     return d;

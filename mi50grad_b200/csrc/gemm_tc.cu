@@ -76,7 +76,9 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
     const int S = p.stages;
     const int t0 = blockIdx.y * p.t_tile;
     const int Tp = (min(p.t_tile, p.T - t0) + 15) & ~15;          // token columns of this CTA
-    const int boxes = (Tp + 63) / 64;
+    // (a CTA pair multiplies whole 256-token operand tiles: rows beyond T are zero-filled by the loads)
+    const int Tm = PAIR ? (Tp + 255) & ~255 : Tp;
+    const int box = p.box_rows, boxes = (Tp + box - 1) / box;     // token rows per TMA load
     // (CTA pairs: a CTA stages only its half of the token rows)
     const int b_stage_bytes = ((p.t_tile + 63) / 64) * 64 * 128 / (PAIR ? 2 : 1);
     // MH = 2: the CTA owns 256 outputs as two M = 128 accumulators that share every activation tile (half the
@@ -104,7 +106,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
     uint4* wring = (uint4*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);   // [TC_RING][2][512 producer threads]: 16 B of nibbles, 2 x 8 B scale/zero
 
     int tmem_cols = 32;
-    while (tmem_cols < Tp) tmem_cols <<= 1;
+    while (tmem_cols < Tm) tmem_cols <<= 1;
     if (MH == 2) tmem_cols = 512;                  // accumulator h at column 256 h (Tp <= 256)
 
     if (tid == 0) {
@@ -231,10 +233,18 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
         }
         cp_async_wait<0>();
         // ================= epilogue =================
-        if (ok) ok = mbar_wait(acc_full, 0, abort_flag);
+        // (one lane polls, the other epilogue warps sleep at a hardware barrier: with dense weights they have
+        // nothing else to do, and hundreds of polling threads slow the TMA and MMA warps down)
+        if (warp == 0) {
+            if (lane == 0 && ok) mbar_wait(acc_full, 0, abort_flag);
+            __syncwarp();
+        }
+        asm volatile("bar.sync 1, %0;" :: "n"(TC_PRODUCERS * 32) : "memory");
+        ok = ok && !*abort_flag;
         tc_fence_after();
         if (ok) {
             const int lg = warp & 3;               // tensor-memory lane group this warp may read
+            const size_t plane = (size_t)blockIdx.z * (size_t)p.plane_stride;     // (split-K of TC_EPI_STORE_F32)
             for (int hc = 0; hc < MH; ++hc)
             for (int c0 = (warp >> 2) * 32; c0 < Tp; c0 += (TC_PRODUCERS / 4) * 32) {
                 const int n = blockIdx.x * (TC_BM * MH) + hc * TC_BM + lg * 32 + lane;
@@ -273,7 +283,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                             float v = __uint_as_float(r[c]);
                             size_t o = (size_t)tt * p.ldo + n;
                             if (p.epi == TC_EPI_STORE_F16) tc_store16(p, o, v);
-                            else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
+                            else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o + plane] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
                             else if (gridDim.z > 1) atomicAdd((float*)p.out + o, v);     // split-K partial
                             else ((float*)p.out)[o] += v;
                         }
@@ -285,25 +295,26 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
         // ================= activation producer (TMA) =================
         {
             const bool dense = p.dense != 0;
+            const int spins = dense ? 64 : 0;
             // pair mode: of every 256-token operand tile this CTA loads rows [128 crank, 128 crank + 128)
-            const uint32_t tx = (pair ? (uint32_t)(Tp / 2) * 128u : (uint32_t)boxes * 64 * 128) + (dense ? (uint32_t)a_bytes : 0u);
+            const uint32_t tx = (pair ? (uint32_t)(Tm / 2) * 128u : (uint32_t)(boxes * box) * 128u) + (dense ? (uint32_t)a_bytes : 0u);
             const int row_w = blockIdx.x * (TC_BM * MH);
             int st = 0;
             uint32_t ph = 0;
             unsigned char* a = sA;
             unsigned char* b = sB;
             for (int kb = 0, kx = kb_lo * TC_BK; kb < KB; ++kb, kx += TC_BK) {
-                if (!mbar_wait(&empty[st], ph ^ 1, abort_flag)) break;
+                if (!mbar_wait(&empty[st], ph ^ 1, abort_flag, spins)) break;
                 if (elect_one()) {
                     mbar_arrive_expect_tx(&full[st], tx);
                     if (dense) for (int hc = 0; hc < MH; ++hc) tma_load_2d(a + hc * TC_A_BYTES, &wmap, kx, row_w + hc * TC_BM, &full[st]);
                     if (pair) {
-                        for (int j = 0; j < Tp / 256; ++j)
+                        for (int j = 0; j < Tm / 256; ++j)
                             for (int bx = 0; bx < 2; ++bx)
                                 tma_load_2d(b + j * (128 * 128) + bx * (64 * 128), &xmap, kx, t0 + j * 256 + (int)crank * 128 + bx * 64, &full[st]);
                     } else {
                         for (int bx = 0; bx < boxes; ++bx)
-                            tma_load_2d(b + bx * (64 * 128), &xmap, kx, t0 + bx * 64, &full[st]);
+                            tma_load_2d(b + bx * (box * 128), &xmap, kx, t0 + bx * box, &full[st]);
                     }
                 }
                 __syncwarp();
@@ -314,7 +325,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
     } else {
         // ================= MMA issuer =================
         {
-            const bool dense = p.dense != 0;
+            const int spins = p.dense ? 64 : 0;
             const int n1 = min(Tp, 256), n2 = Tp - n1;
             const uint32_t fmt = p.bf16 ? TC_IDESC_BF16 : 0u;
             const uint32_t idesc1 = make_idesc_f16(n1) | fmt, idesc2 = make_idesc_f16(n2 > 0 ? n2 : 16) | fmt;
@@ -326,10 +337,10 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
             int st = 0;
             uint32_t ph = 0;
             bool ok = true;
-            const uint32_t idesc_pair = make_idesc_f16_m256(256);
+            const uint32_t idesc_pair = make_idesc_f16_m256(256) | fmt;
             const uint64_t b_pair_half = (128 * 128) >> 4;
             for (int kb = 0; kb < KB; ++kb) {
-                ok = mbar_wait(&full[st], ph, abort_flag);
+                ok = mbar_wait(&full[st], ph, abort_flag, spins);
                 if (!ok) break;
                 if constexpr (PAIR) {
                     if (crank != 0) {
@@ -347,7 +358,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                     if (elect_one()) {
 #pragma unroll
                         for (int k16 = 0; k16 < TC_BK / 16; ++k16)
-                            for (int j = 0; j < Tp / 256; ++j)
+                            for (int j = 0; j < Tm / 256; ++j)
                                 tc_mma_f16_pair(tmem_base + 256 * j, ad + 2 * k16, bd + j * b_pair_half + 2 * k16, idesc_pair, (kb | k16) ? 1u : 0u);
                         tc_commit_pair(&empty[st]);
                     }
@@ -406,7 +417,9 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
     CUtensorMap map;
     cuuint64_t dims[2] = {(cuuint64_t)p->K, (cuuint64_t)p->T};
     cuuint64_t strides[1] = {(cuuint64_t)ldx * 2};
-    cuuint32_t box[2] = {TC_BK, 64};
+    // (as few loads per k-block as a box of at most 256 rows allows; a CTA's stage holds t_tile rounded up to 64)
+    const int box_rows = p->cta_pair ? 64 : (p->t_tile <= 256 ? (p->t_tile + 63) / 64 * 64 : (p->t_tile % 256 ? 64 : 256));
+    cuuint32_t box[2] = {TC_BK, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     const CUtensorMapDataType dtype = p->bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
     CUresult r = enc(&map, dtype, 2, (void*)x, dims, strides, box, estr,
@@ -424,14 +437,17 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
         if (r != CUDA_SUCCESS) return cudaErrorInvalidValue;
     }
     GemmTcParams q = *p;
+    q.box_rows = box_rows;
     q.dense = w ? 1 : 0;
     // 256-output tiles: only with at most 256 tokens per CTA (two accumulators of 256 columns) and a matrix that
     // is a whole number of such tiles
     if (q.m_halves == 2 && (q.t_tile > 256 || (q.NTL * 16) % (2 * TC_BM) != 0)) q.m_halves = 1;
     if (q.m_halves != 2) q.m_halves = 1;
     dim3 grid(q.NTL * 16 / (TC_BM * q.m_halves), (q.T + q.t_tile - 1) / q.t_tile, 1);
-    // CTA pairs: whole 256-token operand tiles only, an even number of output tiles, 128-output CTAs
-    if (q.cta_pair && (q.m_halves != 1 || (grid.x & 1) || (q.t_tile != 256 && q.t_tile != 512) || q.T % q.t_tile != 0)) q.cta_pair = 0;
+    // CTA pairs: 256-token operand tiles, an even number of 128-output CTAs (with dense weights a surplus tile
+    // is made up: its rows are zero-filled and not stored)
+    if (q.cta_pair && q.dense && q.m_halves == 1) grid.x += grid.x & 1;
+    if (q.cta_pair && (q.m_halves != 1 || (grid.x & 1) || (q.t_tile != 256 && q.t_tile != 512))) q.cta_pair = 0;
     size_t per_stage = (size_t)q.m_halves * TC_A_BYTES + (size_t)((q.t_tile + 63) / 64) * 64 * 128 / (q.cta_pair ? 2 : 1);
     // as many stages as shared memory holds next to the weight ring, an even number (the two producer
     // groups alternate stages); deep pipelines matter most for few tokens, where a stage is consumed quickly
@@ -446,7 +462,8 @@ static int launch_tc(const GemmTcParams* p, const void* w, int ldw, int n_rows_w
         cudaError_t e = optin.ensure(gemm_int4_tc_kernel<false>, smem);
         if (e != cudaSuccess) return e;
     }
-    int ks = (q.epi == TC_EPI_RESID_F32 && q.k_splits > 1) ? q.k_splits : 1;
+    const bool planes = q.epi == TC_EPI_STORE_F32 && q.plane_stride > 0 && q.softcap <= 0.f;
+    int ks = ((q.epi == TC_EPI_RESID_F32 || planes) && q.k_splits > 1) ? q.k_splits : 1;
     if (ks > q.KB) ks = q.KB;
     if (ks > 1) { const int per = (q.KB + ks - 1) / ks; ks = (q.KB + per - 1) / per; }     // no empty split
     grid.z = ks;

@@ -29,15 +29,24 @@ struct GemmTcParams {
     long long part_stride;       // floats between the two parity halves of a staging buffer
     int push_tp, push_rank;
     unsigned int push_per;       // float4 elements per slice
-    int k_splits;                // TC_EPI_RESID_F32 only: CTAs along K per output tile (grid z); their partial
-                                 // products are added to out with atomic adds (0 or 1: no split)
+    int k_splits;                // CTAs along K per output tile (grid z; 0 or 1: no split).  TC_EPI_RESID_F32: their
+                                 // partial products are added to out with atomic adds; TC_EPI_STORE_F32 with
+                                 // plane_stride: split z stores its own plane, which the consumer sums
+                                 // (b2_gemm_tc_splits gives the number of planes)
     int cta_pair;                // 1: adjacent output tiles run as CTA pairs (cta_group::2 MMAs, M = 256 over two SMs); needs
-                                 // 128-output CTAs, t_tile 256 or 512 dividing T, an even number of output tiles
+                                 // 128-output CTAs, t_tile 256 or 512, and (INT4 weights) an even number of output tiles
     int bf16;                // 1 (dense weights only): operands and 16-bit outputs are bf16 instead of fp16
     float softcap;           // TC_EPI_STORE_F32: > 0 stores softcap * tanh(y / softcap)
+    long long plane_stride;  // floats between the planes of a split-K TC_EPI_STORE_F32
+    int box_rows;            // set by the launcher: token rows per TMA load
     int pad3;
 };
 
+// planes a launch with `want` splits over K columns leaves (no split is empty)
+static inline int b2_gemm_tc_splits(int K, int want) {
+    const int KB = (K + 63) / 64, ks = want < 1 ? 1 : (want > KB ? KB : want), per = (KB + ks - 1) / ks;
+    return (KB + per - 1) / per;
+}
 
 B2_API int b2_gemm_int4_tc(const GemmTcParams* p, const void* x, int ldx, cudaStream_t stream);
 B2_API int b2_gemm_f16_tc(const GemmTcParams* p, const void* w, int ldw, const void* x, int ldx, cudaStream_t stream);

@@ -51,11 +51,12 @@ struct DenseGemvParams {
     void* out;
     float* ss_out;           // DG_STORE_F32, optional: [rows][ss_np], entry of CTA i = sum over its outputs
     int ldw, ldx, K, N, rows, ldo, mode, dt;
-    int rpc;                 // outputs per CTA: 8, 16 or 32 (DG_SILU_PAIR: 16 or 32)
+    int rpc;                 // outputs per CTA, see b2_gemv_dense
     int ss_np;
     float softcap;
-    int pad;
+    int mma;                 // 1: tensor-core kernel for any number of bf16 rows
 };
+#define DG_FMA_ROWS 2        // bf16 rows up to which the FMA kernel serves
 
 // ---- many-row projection in fp32 (csrc/gemm_f32.cu); same epilogues
 struct GemmF32Params {
@@ -105,7 +106,7 @@ B2_API int b2_gemm_f32(const GemmF32Params* p, cudaStream_t s);
 B2_API int b2_embed_rows(const void* embed, const int* row_tokens, const void* rows, const void* seqs, float* h, void* xb,
                          int ldx, int n_rows, int H, int vocab, int dt, cudaStream_t s);
 B2_API int b2_post_norm(float* h, const float* m, const float* w, const float* final_w, void* xb, int ldx, int n_rows, int H,
-                        float eps, int dt, cudaStream_t s);
+                        float eps, int dt, int planes, long long plane_stride, cudaStream_t s);
 B2_API int b2_mix_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s);
 B2_API int b2_window_attn_decode(const MixLayer* l, const MixRun* r, cudaStream_t s);
 B2_API int b2_window_attn_rows(const MixLayer* l, const MixRun* r, cudaStream_t s);

@@ -31,7 +31,8 @@ B2_API int b2_embed_rows(const void* embed, const int* row_tokens, const void* r
 // VEC: H % 4 == 0, H <= 8192 and ldx % 4 == 0, the row stays in registers between its passes
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) post_norm_kernel(float* __restrict__ h, const float* __restrict__ m, const float* __restrict__ w,
-                                                        const float* __restrict__ fw, T* __restrict__ xb, int ldx, int H, float eps) {
+                                                        const float* __restrict__ fw, T* __restrict__ xb, int ldx, int H, float eps, int planes,
+                                                        size_t plane_stride) {
     __shared__ float red[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -47,6 +48,8 @@ __global__ void __launch_bounds__(256) post_norm_kernel(float* __restrict__ h, c
             const int i = tid + 256 * u;
             a[u] = make_float4(0.f, 0.f, 0.f, 0.f); x[u] = a[u];
             if (i < n4) { x[u] = ((const float4*)hr)[i]; if (mr) a[u] = ((const float4*)mr)[i]; }
+            for (int q = 1; q < planes; ++q)
+                if (i < n4) { const float4 b = *(const float4*)(mr + q * plane_stride + 4 * i); a[u].x += b.x; a[u].y += b.y; a[u].z += b.z; a[u].w += b.w; }
             ss += a[u].x * a[u].x + a[u].y * a[u].y + a[u].z * a[u].z + a[u].w * a[u].w;
         }
         if (mr) {
@@ -83,16 +86,17 @@ __global__ void __launch_bounds__(256) post_norm_kernel(float* __restrict__ h, c
             }
         }
     } else {
+        auto sum = [&](int i) { float v = mr[i]; for (int q = 1; q < planes; ++q) v += mr[q * plane_stride + i]; return v; };
         float inv = 0.f;
         if (mr) {
             float ss = 0.f;
-            for (int i = tid; i < H; i += 256) ss += mr[i] * mr[i];
+            for (int i = tid; i < H; i += 256) { const float v = sum(i); ss += v * v; }
             inv = rsqrtf(block_sum(ss, red) / (float)H + eps);
         }
         float ss = 0.f;
         for (int i = tid; i < H; i += 256) {                 // (a thread re-reads only what it wrote)
             float v = hr[i];
-            if (mr) { v += mr[i] * inv * w[i]; hr[i] = v; }
+            if (mr) { v += sum(i) * inv * w[i]; hr[i] = v; }
             ss += v * v;
         }
         float fin = 1.f;
@@ -101,14 +105,16 @@ __global__ void __launch_bounds__(256) post_norm_kernel(float* __restrict__ h, c
     }
 }
 
-// h += rmsnorm(m) * w (m null: h as it is), then xb = h, or with final_w xb = rmsnorm(h) * final_w.
+// h += rmsnorm(m) * w (m null: h as it is), then xb = h, or with final_w xb = rmsnorm(h) * final_w.  m is the sum
+// of `planes` arrays plane_stride floats apart (the splits of a projection over K).
 B2_API int b2_post_norm(float* h, const float* m, const float* w, const float* final_w, void* xb, int ldx, int n_rows, int H,
-                        float eps, int dt, cudaStream_t s) {
-    const bool vec = (H & 3) == 0 && H <= 8192 && (ldx & 3) == 0;
+                        float eps, int dt, int planes, long long plane_stride, cudaStream_t s) {
+    if (!m) planes = 1;
+    const bool vec = (H & 3) == 0 && H <= 8192 && (ldx & 3) == 0 && (plane_stride & 3) == 0;
     if (dt == DT_BF16) {
-        if (vec) return launch_pdl(post_norm_kernel<bf16, true>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (bf16*)xb, ldx, H, eps);
-        return launch_pdl(post_norm_kernel<bf16, false>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (bf16*)xb, ldx, H, eps);
+        if (vec) return launch_pdl(post_norm_kernel<bf16, true>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (bf16*)xb, ldx, H, eps, planes, (size_t)plane_stride);
+        return launch_pdl(post_norm_kernel<bf16, false>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (bf16*)xb, ldx, H, eps, planes, (size_t)plane_stride);
     }
-    if (vec) return launch_pdl(post_norm_kernel<float, true>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (float*)xb, ldx, H, eps);
-    return launch_pdl(post_norm_kernel<float, false>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (float*)xb, ldx, H, eps);
+    if (vec) return launch_pdl(post_norm_kernel<float, true>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (float*)xb, ldx, H, eps, planes, (size_t)plane_stride);
+    return launch_pdl(post_norm_kernel<float, false>, dim3(n_rows), dim3(256), 0, s, h, m, w, final_w, (float*)xb, ldx, H, eps, planes, (size_t)plane_stride);
 }

@@ -33,8 +33,12 @@ __device__ __forceinline__ bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
 // Bounded wait.  Returns false (and raises *abort_flag) when the time budget is exhausted or
 // another role has already given up.  The timer read between polls also acts as a back-off:
 // polling the barrier harder was measured to slow the pipeline down.
-__device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
+// `spins`: polls before the timer is read at all (for waits that are short and have a single poller).
+__device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int spins = 0) {
     if (mbar_try_wait(bar, parity)) return true;
+#pragma unroll 1
+    for (int i = 0; i < spins; ++i)
+        if (mbar_try_wait(bar, parity)) return true;
     long long t0 = globaltimer_ns();
     for (;;) {
 #pragma unroll 1

@@ -37,13 +37,13 @@ def _up8(n: int) -> int:
     return -(-n // 8) * 8
 
 
-def gemv_outputs_per_cta(n: int, pair: bool = False) -> int:
-    """Outputs per CTA of a decode projection with n outputs: as many as leave every SM about two CTAs
-    (a gate / up pair needs at least 16)."""
+def gemv_outputs_per_cta(n: int, tensor_core: bool, pair: bool = False) -> int:
+    """Outputs per CTA of a decode projection with n outputs: as many as leave every SM about one and a half
+    CTAs (the tensor-core kernel takes at least 16, the other at least 8, a gate / up pair at least 16)."""
     for r in (32, 16):
-        if n >= r * 2 * 148:
+        if n >= r * 222:
             return r
-    return 16 if pair else 8
+    return 16 if tensor_core or pair else 8
 
 
 class MixerLinear:
@@ -51,13 +51,16 @@ class MixerLinear:
 
     def __init__(self, w: torch.Tensor, kind: int, dtype: torch.dtype, device, pair: bool = False):
         self.N, self.K = w.shape
-        self.kind, self.rpc = kind, gemv_outputs_per_cta(self.N, pair)
+        self.kind = kind
+        self.rpc_few = gemv_outputs_per_cta(self.N, False, pair)         # one or two rows, and fp32
+        self.rpc = gemv_outputs_per_cta(self.N, True) if kind == L.LIN_BF16 else self.rpc_few
         self.w = torch.zeros(self.N, _up8(self.K), dtype=dtype, device=device)
         self.w[:, :self.K].copy_(w)
 
     def desc(self) -> L.LinearDesc:
         d = L.LinearDesc()
-        d.kind, d.K, d.N, d.L, d.ldw, d.w = self.kind, self.K, self.N, self.rpc, self.w.shape[1], self.w.data_ptr()
+        d.kind, d.K, d.N, d.ldw, d.w = self.kind, self.K, self.N, self.w.shape[1], self.w.data_ptr()
+        d.L, d.kslice = self.rpc, self.rpc_few
         return d
 
     def nbytes(self) -> int:
@@ -218,7 +221,8 @@ class MixerEngine(InferenceEngine):
         b["logits"] = f32(R, b["ld_logits"])
         self.np = -(-H // 8)                                   # one partial sum per CTA of at least 8 outputs
         b["ss"] = f32(R, self.np)
-        b["p_h"], b["p_m"], b["p_xn"] = f32(P, H), f32(P, H), elt(P, ld_x)
+        M_PLANES = 4                                           # splits over K of a many-row output projection
+        b["p_h"], b["p_m"], b["p_xn"] = f32(P, H), f32(M_PLANES, P, H), elt(P, ld_x)
         b["p_proj"], b["p_attn"], b["p_act"] = elt(P, b["ld_proj"]), elt(P, b["ld_attn"]), elt(P, ld_act)
         M = max(P, R)
         b["qbuf"] = elt(M, max(m.H * m.dp for m in mix))
@@ -251,6 +255,7 @@ class MixerEngine(InferenceEngine):
         x = L.MixerModelDesc()
         x.final_norm, x.softcap, x.dt = self.final_norm.data_ptr(), cfg.logit_softcap, self.dt
         x.ss_np, x.ld_x, x.ld_xbc, x.ld_dt, x.ld_u, x.ld_act, x.scratch_rows = self.np, ld_x, ld_xbc, ld_dt, ld_u, ld_act, SR
+        x.m_planes = M_PLANES
         for k in ("m", "p_m", "qbuf", "xbc", "dtb", "ubuf", "attn_scratch", "attn_counters", "ssd_counters", "chunk_state",
                   "chunk_prev", "chunk_decay"):
             if k in b:

@@ -533,10 +533,14 @@ def post_norm_input(h: torch.Tensor, m: Optional[torch.Tensor] = None, w: Option
 
 
 def gemv_dense(lin, x: Optional[torch.Tensor], out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0,
-               pn: Optional[L.PostNorm] = None, rows: Optional[int] = None, ss_out: Optional[torch.Tensor] = None):
-    """1..8 rows times a `MixerLinear`-like object (.w [N][ldw], .K, .N, .rpc); bf16 or fp32."""
+               pn: Optional[L.PostNorm] = None, rows: Optional[int] = None, ss_out: Optional[torch.Tensor] = None, mma: bool = False):
+    """1..8 rows times a `MixerLinear`-like object (.w [N][ldw], .K, .N, .rpc_few, .rpc); bf16 or fp32.
+    mma: the tensor-core kernel also for one or two bf16 rows."""
     p = L.DenseGemvParams()
-    p.w, p.ldw, p.K, p.N, p.rpc, p.dt = lin.w.data_ptr(), lin.w.stride(0), lin.K, lin.N, lin.rpc, _dt(lin.w)
+    n = rows if x is None else x.shape[0]
+    tc = lin.w.dtype == torch.bfloat16 and (mma or n > L.DG_FMA_ROWS)
+    p.w, p.ldw, p.K, p.N, p.dt, p.mma = lin.w.data_ptr(), lin.w.stride(0), lin.K, lin.N, _dt(lin.w), int(mma)
+    p.rpc = lin.rpc if tc else lin.rpc_few
     if x is not None:
         p.x, p.ldx, p.rows = x.data_ptr(), x.stride(0), x.shape[0]
     else:
@@ -559,17 +563,19 @@ def gemm_f32(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, mode: int = L.
 
 def post_norm_(h: torch.Tensor, m: Optional[torch.Tensor], w: Optional[torch.Tensor], xb: torch.Tensor, eps: float,
                final_w: Optional[torch.Tensor] = None):
-    """h += rmsnorm(m) * w in place; xb = h, or rmsnorm(h) * final_w."""
+    """h += rmsnorm(m) * w in place; xb = h, or rmsnorm(h) * final_w.  A three-dimensional m is summed over its
+    first axis (the planes of a projection split over K)."""
+    planes, stride = (m.shape[0], m.stride(0)) if m is not None and m.dim() == 3 else (1, 0)
     vp = lambda t: C.c_void_p(L.ptr(t))
     L.check(L.lib().b2_post_norm(vp(h), vp(m), vp(w), vp(final_w), vp(xb), xb.stride(0), h.shape[0], h.shape[1], C.c_float(eps),
-                                 _dt(xb), L.stream()), "post_norm")
+                                 _dt(xb), planes, C.c_longlong(stride), L.stream()), "post_norm")
     return h
 
 
 def gemm_bf16_tc(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, epi: int = L.TC_EPI_STORE_F32,
-                 t_tile: Optional[int] = None, softcap: float = 0.0):
+                 t_tile: Optional[int] = None, softcap: float = 0.0, cta_pair: bool = False, k_splits: int = 1):
     """out[t][n] (epi) = x[t] . w[n] for bf16 operands on the tcgen05 tensor cores; any K (row strides
-    multiples of 8)."""
+    multiples of 8).  k_splits > 1: out is [planes][T][N] fp32, the product is the sum of its planes."""
     T, dev = x.shape[0], x.device
     st = _tc_status.get(dev)
     if st is None:
@@ -577,7 +583,8 @@ def gemm_bf16_tc(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, epi: int =
     p = L.GemmTcParams()
     p.K, p.T, p.t_tile, p.epi = x.shape[1], T, t_tile or min(256, -(-T // 16) * 16), epi
     p.n_valid = w.shape[0] // 2 if epi == L.TC_EPI_SILU_PAIR else w.shape[0]
-    p.ldo, p.out, p.status, p.bf16, p.softcap = out.stride(0), out.data_ptr(), st.data_ptr(), 1, softcap
+    p.ldo, p.out, p.status, p.bf16, p.softcap = out.stride(-2), out.data_ptr(), st.data_ptr(), 1, softcap
+    p.cta_pair, p.k_splits, p.plane_stride = int(cta_pair), k_splits, out.stride(0) if out.dim() == 3 else 0
     L.check(L.lib().b2_gemm_f16_tc(C.byref(p), C.c_void_p(w.data_ptr()), w.stride(0), C.c_void_p(x.data_ptr()),
                                    x.stride(0), L.stream()), "gemm_bf16_tc")
     return out

@@ -27,7 +27,7 @@ FIN_NO_COMM, FIN_NO_H_WRITE, FIN_SAVE_EXTRA, FIN_ADD_EXTRA, FIN_NO_NORM = 1, 2, 
 FIN_TEST_WITHHOLD_SIGNAL = 32
 LIN_INT4, LIN_F16, LIN_NONE, LIN_BF16, LIN_F32 = 0, 1, 2, 3, 4
 DT_BF16, DT_F32 = 0, 1
-DG_STORE, DG_SILU_PAIR, DG_STORE_F32 = 0, 1, 2
+DG_STORE, DG_SILU_PAIR, DG_STORE_F32, DG_FMA_ROWS = 0, 1, 2, 2
 STEP_EMBED_TOKENS, STEP_LM_HEAD, STEP_ARGMAX, STEP_ADVANCE, STEP_NO_COMMIT_DELTA = 1, 2, 4, 8, 16
 STEP_MATERIALIZE_XN = 32
 STEP_SPEC, STEP_GEMM_PATH, STEP_HEAD_LAST = 64, 128, 256
@@ -119,7 +119,8 @@ class GemmTcParams(C.Structure):
                 ("gshift", i32), ("T", i32), ("t_tile", i32), ("n_valid", i32), ("ldo", i32), ("epi", i32),
                 ("stages", i32), ("out", vp), ("status", vp), ("m_halves", i32), ("dense", i32),
                 ("push", vp * MAX_TP), ("epoch", vp), ("part_stride", i64), ("push_tp", i32), ("push_rank", i32),
-                ("push_per", C.c_uint), ("k_splits", i32), ("cta_pair", i32), ("bf16", i32), ("softcap", f32), ("pad3", i32)]
+                ("push_per", C.c_uint), ("k_splits", i32), ("cta_pair", i32), ("bf16", i32), ("softcap", f32),
+                ("plane_stride", i64), ("box_rows", i32), ("pad3", i32)]
 
 
 TC_EPI_STORE_F16, TC_EPI_SILU_PAIR, TC_EPI_STORE_F32, TC_EPI_RESID_F32 = 0, 1, 2, 3
@@ -210,7 +211,7 @@ class PostNorm(C.Structure):
 class DenseGemvParams(C.Structure):
     _fields_ = [("w", vp), ("x", vp), ("pn", PostNorm), ("out", vp), ("ss_out", vp), ("ldw", i32), ("ldx", i32), ("K", i32),
                 ("N", i32), ("rows", i32), ("ldo", i32), ("mode", i32), ("dt", i32), ("rpc", i32), ("ss_np", i32),
-                ("softcap", f32), ("pad", i32)]
+                ("softcap", f32), ("mma", i32)]
 
 
 class GemmF32Params(C.Structure):
@@ -243,7 +244,7 @@ class MixerLayerDesc(C.Structure):
 
 class MixerModelDesc(C.Structure):
     _fields_ = [("layers", vp), ("final_norm", vp), ("softcap", f32), ("dt", i32), ("ss_np", i32), ("ld_x", i32),
-                ("ld_xbc", i32), ("ld_dt", i32), ("ld_u", i32), ("ld_act", i32), ("scratch_rows", i32), ("pad", i32),
+                ("ld_xbc", i32), ("ld_dt", i32), ("ld_u", i32), ("ld_act", i32), ("scratch_rows", i32), ("m_planes", i32),
                 ("m", vp), ("p_m", vp), ("qbuf", vp), ("xbc", vp), ("dtb", vp), ("ubuf", vp),
                 ("attn_scratch", vp), ("attn_counters", vp), ("ssd_counters", vp),
                 ("chunk_state", vp), ("chunk_prev", vp), ("chunk_decay", vp)]

@@ -109,7 +109,8 @@ def test_gate_up_interleave():
         want = (g[j], u[j]) if j < 19 else (torch.zeros(6), torch.zeros(6))
         assert torch.equal(w[r], want[0]) and torch.equal(w[r + 8], want[1])
     for n in (1, 7, 500, 5000, 50000, 200000):
-        assert gemv_outputs_per_cta(n) in (8, 16, 32) and gemv_outputs_per_cta(n, True) >= 16
+        assert gemv_outputs_per_cta(n, True) in (16, 32, 64, 128)
+        assert gemv_outputs_per_cta(n, False) in (8, 16, 32) and gemv_outputs_per_cta(n, False, True) in (16, 32)
 
 
 @pytest.mark.parametrize("name", ["mixed", "odd_width"])

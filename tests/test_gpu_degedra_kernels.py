@@ -26,14 +26,16 @@ def _lin(w, dtype, rpc):
     N, K = w.shape
     d = torch.zeros(N, -(-K // 8) * 8, dtype=dtype, device="cuda")
     d[:, :K] = w
-    return SimpleNamespace(w=d, N=N, K=K, rpc=rpc)
+    few = min(rpc, 32)
+    return SimpleNamespace(w=d, N=N, K=K, rpc=max(16, rpc) if dtype == torch.bfloat16 else few, rpc_few=few)
 
 
 # ------------------------------------------------------------------ projections
 @pytest.mark.parametrize("dt", ["bf16", "f32"])
-@pytest.mark.parametrize("N,K,rows,rpc", [(37, 90, 1, 8), (64, 200, 3, 16), (301, 2056, 8, 32), (1000, 5000, 2, 8),
-                                          (40, 17000, 8, 16), (129, 4096, 5, 32)])
-def test_gemv_dense(dt, N, K, rows, rpc):
+@pytest.mark.parametrize("mma", [False, True])
+@pytest.mark.parametrize("N,K,rows,rpc", [(37, 90, 1, 8), (333, 5000, 2, 128), (64, 200, 3, 16), (301, 2056, 8, 32), (1000, 5000, 2, 8),
+                                          (40, 17000, 8, 16), (129, 4096, 5, 32), (700, 1500, 7, 64)])
+def test_gemv_dense(dt, N, K, rows, rpc, mma):
     from mi50grad_b200.ops import kernels as K_
     from mi50grad_b200.ops import lib as L
     T, _, tol = DTS[dt]
@@ -45,19 +47,20 @@ def test_gemv_dense(dt, N, K, rows, rpc):
     xin = xs[:, :K]
     out = torch.full((rows, N), 7.0, device="cuda")
     ss = torch.zeros(rows, -(-N // 8), device="cuda")
-    K_.gemv_dense(lin, xin, out, L.DG_STORE_F32, ss_out=ss)
+    K_.gemv_dense(lin, xin, out, L.DG_STORE_F32, ss_out=ss, mma=mma)
     _close(out, ref, 2e-5)
     assert torch.allclose(ss.sum(1), out.pow(2).sum(1), rtol=1e-4)
-    K_.gemv_dense(lin, xin, out, L.DG_STORE_F32, softcap=1.5)
+    K_.gemv_dense(lin, xin, out, L.DG_STORE_F32, softcap=1.5, mma=mma)
     _close(out, 1.5 * torch.tanh(ref / 1.5), 2e-5)
     o16 = torch.zeros(rows, N, dtype=T, device="cuda")
-    K_.gemv_dense(lin, xin, o16, L.DG_STORE)
+    K_.gemv_dense(lin, xin, o16, L.DG_STORE, mma=mma)
     _close(o16, ref, tol)
 
 
 @pytest.mark.parametrize("dt", ["bf16", "f32"])
-@pytest.mark.parametrize("H,rows", [(90, 3), (256, 8), (5000, 1)])
-def test_gemv_dense_forms_the_residual_update(dt, H, rows):
+@pytest.mark.parametrize("mma", [False, True])
+@pytest.mark.parametrize("H,rows", [(90, 3), (256, 8), (5000, 1), (168, 2)])
+def test_gemv_dense_forms_the_residual_update(dt, H, rows, mma):
     from mi50grad_b200.ops import kernels as K_
     from mi50grad_b200.ops import lib as L
     T, _, tol = DTS[dt]
@@ -70,11 +73,11 @@ def test_gemv_dense_forms_the_residual_update(dt, H, rows):
     ss = torch.stack([c.pow(2).sum(1) for c in md.split(-(-H // parts), dim=1)], 1).contiguous()
     out = torch.zeros(rows, 48, device="cuda")
     pn = K_.post_norm_input(hd, md, wd, ss, hout, 1e-5)
-    K_.gemv_dense(_lin(w, T, 16), None, out, L.DG_STORE_F32, pn=pn, rows=rows)
+    K_.gemv_dense(_lin(w, T, 16), None, out, L.DG_STORE_F32, pn=pn, rows=rows, mma=mma)
     _close(hout, x, 2e-6)
     assert torch.equal(hd.cpu(), h)
     _close(out, x.to(T).double() @ w.double().T, tol)
-    K_.gemv_dense(_lin(w, T, 8), None, out, L.DG_STORE_F32, pn=K_.post_norm_input(hd), rows=rows)
+    K_.gemv_dense(_lin(w, T, 8), None, out, L.DG_STORE_F32, pn=K_.post_norm_input(hd), rows=rows, mma=mma)
     _close(out, h.to(T).double() @ w.double().T, tol)
 
 
@@ -127,6 +130,31 @@ def test_many_row_gemms(N, K, T_):
     K_.gemm_tc_check_status()
 
 
+@pytest.mark.parametrize("N,K,T_,t", [(640, 1032, 130, 256), (129, 4096, 511, 512), (900, 512, 512, 512), (384, 640, 300, 256)])
+def test_gemm_cta_pairs_and_k_splits(N, K, T_, t):
+    """Two-CTA tiles (odd tile counts and ragged token counts too), and products left as planes to be summed."""
+    from mi50grad_b200.ops import kernels as K_
+    from mi50grad_b200.ops import lib as L
+    w, x = _lin(_rnd(N, K, std=K ** -0.5), torch.bfloat16, 8).w, _lin(_rnd(T_, K, seed=1), torch.bfloat16, 8).w
+    w, x = w[:, :K], x[:, :K]
+    ref = x.double().cpu() @ w.double().cpu().T
+    out = torch.zeros(T_, N, device="cuda")
+    K_.gemm_bf16_tc(w, x, out, t_tile=t, cta_pair=True)
+    _close(out, ref, 1e-5)
+    if N % 16 == 0:
+        o16 = torch.zeros(T_, N // 2, dtype=torch.bfloat16, device="cuda")
+        K_.gemm_bf16_tc(w, x, o16, L.TC_EPI_SILU_PAIR, t_tile=t, cta_pair=True)
+        r = ref.reshape(T_, N // 16, 2, 8)
+        _close(o16, (O.silu(r[:, :, 0]) * r[:, :, 1]).reshape(T_, N // 2), 1e-2)
+    for pair in (True, False):
+        for ks in (2, 3):
+            planes = torch.zeros(ks, T_, N, device="cuda")
+            K_.gemm_bf16_tc(w, x, planes, t_tile=t if pair else 128, cta_pair=pair, k_splits=ks)
+            _close(planes.sum(0), ref, 1e-5)
+            assert float(planes[-1].abs().max()) > 0
+    K_.gemm_tc_check_status()
+
+
 @pytest.mark.parametrize("dt", ["bf16", "f32"])
 @pytest.mark.parametrize("H", [90, 168, 4096])
 def test_post_norm(dt, H):
@@ -140,6 +168,10 @@ def test_post_norm(dt, H):
         K_.post_norm_(hd, m.cuda(), w.cuda(), xb, 1e-4, None if fw is None else fw.cuda())
         _close(hd, x, 2e-6)
         _close(xb[:, :H], x if fw is None else O.rms(x, 1e-4) * f.double(), tol)
+        hd = h.cuda()
+        parts = torch.stack([0.25 * m, 0.5 * m, 0.25 * m]).cuda()
+        K_.post_norm_(hd, parts, w.cuda(), xb, 1e-4, None if fw is None else fw.cuda())
+        _close(hd, x, 2e-6)
 
 
 # ------------------------------------------------------------------ the mixer's kernels
