@@ -1,7 +1,8 @@
 """mi50grad_b200: a B200-native tensor-parallel inference engine for the
 Qwen3.5 hybrid (Gated DeltaNet + gated full attention) decoder with INT4
-weight-only quantisation."""
-from .config import (EngineConfig, QwenConfig, kv_cache_bytes, load_config_from_json,
+weight-only quantisation, and for the Degedra decoder (windowed attention beside
+a Mamba-2 recurrence) with bf16 weights."""
+from .config import (DegedraConfig, EngineConfig, QwenConfig, kv_cache_bytes, load_config_from_json,
                      memory_budget, qwen35_27b, tiny_config, QWEN_GEMM_SHAPES)
 
 __version__ = "0.1.0"
@@ -20,6 +21,8 @@ def __getattr__(name):
         "TreeSpeculativeDecoder": ".generate.tree_speculative", "OracleEngine": ".models.oracle",
         "QwenWeightLoader": ".loaders", "AWQWeightLoader": ".loaders", "CompressedTensorsLoader": ".loaders",
         "detect_quant_format": ".loaders", "load_awq_or_gptq": ".loaders",
+        "MixerEngine": ".engine.mixer_engine", "build_engine": ".models.registry", "load_model_config": ".models.registry",
+        "DegedraLoader": ".loaders.mixer",
         "TorchBaselineEngine": ".baseline.torch_engine",
     }
     if name in table:

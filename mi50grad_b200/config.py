@@ -363,6 +363,14 @@ class DegedraConfig:
                    for l in self.layers)
 
 
+def tiny_degedra_config() -> DegedraConfig:
+    """Three small layers, the last one sharing the first one's tensors (smoke runs, examples)."""
+    a = WindowAttentionSpec(heads=6, kv_heads=2, dim=48, rot_dims=32, rot_base=10000.0, scale=48 ** -0.5, window=40)
+    s = SSDSpec(heads=6, vdim=32, state=64, groups=3, conv=4, norm_groups=3)
+    l = ParallelLayerSpec(a, s, 0.9, 0.7, 320)
+    return DegedraConfig(256, 1000, 1e-6, [l, dataclasses.replace(l, ff=0), dataclasses.replace(l, weights_of=0)], 25.0)
+
+
 def degedra_config_from_dict(c: dict) -> DegedraConfig:
     layers = []
     for i, e in enumerate(c["layers"]):

@@ -767,29 +767,21 @@ static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, in
     }
     GemmTcParams p;
     memset(&p, 0, sizeof(p));
-    // Token tile, CTA pairs and K splits: an SM takes in about 65 GB/s of operand tiles (measured, whatever the
-    // tile), so a 64-k block of a 128-output CTA costs the time of its 16 KB of weights and 128 bytes per token
-    // row it loads (half of the rows in a pair), but not less than its tensor time.
-    const int ctas_n = (L.N + 127) / 128, KB = (L.K + 63) / 64;
-    int best_t = 64, best_pair = 0, best_ks = 1;
+    // Token tile and K splits from a fit to measured times (us): a 64-k block of a [128 x t] tile costs about
+    // 0.22 + t / 1000 (the tensor instructions' issue), a tile about 6 + t / 33 outside its k loop, a further
+    // plane 0.7 in its consumer.
+    const int ctas_n = (L.N + 127) / 128, KB = (L.K + 63) / 64, Tr = (T + 15) & ~15;
+    int best_t = 64, best_ks = 1;
     double best = 1e30;
-    const int tiles[] = {64, 96, 128, 160, 192, 224, 256, 512};
-    for (int i = 0; i < 8; ++i)
-        for (int pair = 0; pair < 2; ++pair) {
-            const int t = tiles[i];
-            if (pair ? t < 256 : (t > 256 || t >= T + 64)) continue;
-            if (pair && t == 512 && T <= 256) continue;
-            const int nn = pair ? ctas_n + (ctas_n & 1) : ctas_n, nt = (T + t - 1) / t;
-            const double load = (16384.0 + (pair ? 64.0 : 128.0) * t) / 65000.0, math = t / 256.0 * 0.45;
-            const double blk = load > math ? load : math;
-            for (int ks = 1; ks <= max_ks; ++ks) {
-                const int k1 = b2_gemm_tc_splits(L.K, ks), waves = (nn * nt * k1 + 147) / 148;
-                const double cost = waves * ((KB + k1 - 1) / k1 * blk + 3.0) + (k1 > 1 ? 0.7 * k1 : 0.0);
-                if (cost < best) { best = cost; best_t = t; best_pair = pair; best_ks = ks; }
-            }
+    for (int t = 64; t <= 256; t += 16) {
+        if (t >= Tr + 16) break;
+        for (int ks = 1; ks <= max_ks; ++ks) {
+            const int k1 = b2_gemm_tc_splits(L.K, ks), waves = (ctas_n * ((T + t - 1) / t) * k1 + 147) / 148;
+            const double cost = waves * ((KB + k1 - 1) / k1 * (0.22 + 0.001 * t) + 6.0 + 0.03 * t) + 0.7 * (k1 - 1);
+            if (cost < best - 1e-9) { best = cost; best_t = t; best_ks = ks; }
         }
-    p.K = L.K; p.T = T; p.t_tile = best_t; p.cta_pair = best_pair; p.k_splits = best_ks;
-    if (!best_pair && p.t_tile > ((T + 15) & ~15)) p.t_tile = (T + 15) & ~15;
+    }
+    p.K = L.K; p.T = T; p.t_tile = best_t > Tr ? Tr : best_t; p.k_splits = best_ks;
     p.ldo = ldo; p.out = out; p.status = d->m.tc_status; p.bf16 = 1; p.softcap = softcap;
     if (planes) { *planes = b2_gemm_tc_splits(L.K, best_ks); p.plane_stride = (long long)d->m.max_prefill * ldo; }
     p.n_valid = mode == DG_SILU_PAIR ? L.N / 2 : L.N;

@@ -22,3 +22,15 @@ def test_arguments_and_docstring():
     for key in ('"metric"', '"value"', '"unit"', '"n_gpus"', '"ms_per_step"', '"higher_is_better"', '"scaling"',
                 '"vs_baseline"', '"dtype"', '"data"', '"config"', '"clocks"', '"e2e"', '"gpu_launches"'):
         assert key in src, key
+
+
+def test_degedra_mode_compares_models_of_equal_size():
+    src = open(os.path.join(ROOT, "bench.py")).read()
+    assert '"degedra"' in src and 'default="decode"' in src
+    from mi50grad_b200.bench.degedra import SIZES, degedra_config, hybrid_config
+    for size in SIZES:
+        d, h = degedra_config(size), hybrid_config(size)
+        l = d.layers[0]
+        assert (d.hidden_size, l.ff, len(d.layers), d.vocab_size) == (h.hidden_size, h.intermediate_size, h.num_hidden_layers, h.vocab_size)
+        assert l.attention.heads * l.attention.dim == h.full_attn_q_dim
+        assert l.ssd.inner == h.linear_attn_value_dim
