@@ -242,10 +242,15 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
     pdl_wait();
     const bool in = lane * EPL < L.dp;                       // dp is a multiple of EPL (<= 8): lanes are in or out as a whole
     const int col = lane * EPL;
-    float q[GT][EPL], acc[GT][EPL], m[GT], l[GT];
+    // Scores of WD_KEYS keys x GT heads are summed over the lanes by recursive halving: every step a lane hands
+    // half of its values to its partner and keeps the other half, so afterwards each lane holds ONE finished
+    // score (the value with index lane >> SH) and the soft-max costs one exponential per lane.  The running
+    // maximum and sum of a head live in the lanes of its scores.
+    constexpr int NV = WD_KEYS * GT, SH = NV == 32 ? 0 : NV == 16 ? 1 : NV == 8 ? 2 : 3;
+    const int mykey = (lane >> SH) & (WD_KEYS - 1);
+    float q[GT][EPL], acc[GT][EPL], m_l = -INFINITY, l_l = 0.f;
 #pragma unroll
     for (int h = 0; h < GT; ++h) {
-        m[h] = -INFINITY; l[h] = 0.f;
         WRaw<T, EPL> qv;
         wr_load(qv, (const T*)R.qbuf + ((size_t)r * L.H + kvh * Gq + hb + h) * L.dp + col, in && h < nh);
 #pragma unroll
@@ -270,32 +275,47 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
 #pragma unroll
         for (int i = 0; i < WD_KEYS; ++i) { kk[i] = kn[i]; vv[i] = vn[i]; }
         if (s + WD_WARPS * WD_KEYS < a1) fetch(s + WD_WARPS * WD_KEYS);
-        float d[WD_KEYS][GT];
+        float d[NV];                                         // [head][key]
 #pragma unroll
-        for (int i = 0; i < WD_KEYS; ++i)
+        for (int h = 0; h < GT; ++h)
 #pragma unroll
-            for (int h = 0; h < GT; ++h) {
+            for (int i = 0; i < WD_KEYS; ++i) {
                 float x = 0.f;
+                if (h < nh)
 #pragma unroll
-                for (int e = 0; e < EPL; ++e) x = fmaf(q[h][e], wr_get(kk[i], e), x);
-                d[i][h] = x;
+                    for (int e = 0; e < EPL; ++e) x = fmaf(q[h][e], wr_get(kk[i], e), x);
+                d[h * WD_KEYS + i] = x;
             }
+        int off = 16;
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1)
+        for (int n = NV; n > 1; n >>= 1, off >>= 1) {
+            const bool up = lane & off;
 #pragma unroll
-            for (int i = 0; i < WD_KEYS; ++i)
+            for (int i = 0; i < n / 2; ++i) {
+                const float give = up ? d[i] : d[i + n / 2], keep = up ? d[i + n / 2] : d[i];
+                d[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+            }
+        }
 #pragma unroll
-                for (int h = 0; h < GT; ++h) d[i][h] += __shfl_xor_sync(0xffffffffu, d[i][h], o);
+        for (int o = 16 / NV; o > 0; o >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], o);
+        const float sc = s + mykey * WD_WARPS + warp < a1 ? d[0] : -INFINITY;
+        float mn = sc;
+#pragma unroll
+        for (int o = 1; o < WD_KEYS; o <<= 1) mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, o << SH));
+        mn = fmaxf(mn, m_l);                                 // (the first key of the pass is always inside: finite)
+        const float corr_l = expf(m_l - mn), p_l = expf(sc - mn);
+        float ps = p_l;
+#pragma unroll
+        for (int o = 1; o < WD_KEYS; o <<= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o << SH);
+        l_l = l_l * corr_l + ps;
+        m_l = mn;
 #pragma unroll
         for (int h = 0; h < GT; ++h) {
-            float mn = m[h];
+            if (h >= nh) break;
+            const float corr = __shfl_sync(0xffffffffu, corr_l, (h * WD_KEYS) << SH);
+            float pw[WD_KEYS];
 #pragma unroll
-            for (int i = 0; i < WD_KEYS; ++i) if (s + i * WD_WARPS + warp < a1) mn = fmaxf(mn, d[i][h]);
-            const float corr = expf(m[h] - mn);              // (the first key of the pass is always inside: mn is finite)
-            float ps = 0.f, pw[WD_KEYS];
-#pragma unroll
-            for (int i = 0; i < WD_KEYS; ++i) { pw[i] = s + i * WD_WARPS + warp < a1 ? expf(d[i][h] - mn) : 0.f; ps += pw[i]; }
-            l[h] = l[h] * corr + ps;
+            for (int i = 0; i < WD_KEYS; ++i) pw[i] = __shfl_sync(0xffffffffu, p_l, (h * WD_KEYS + i) << SH);
 #pragma unroll
             for (int e = 0; e < EPL; ++e) {
                 float a = acc[h][e] * corr;
@@ -303,12 +323,10 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
                 for (int i = 0; i < WD_KEYS; ++i) a = fmaf(pw[i], wr_get(vv[i], e), a);
                 acc[h][e] = a;
             }
-            m[h] = mn;
         }
     }
     // ---- merge the warps, one head at a time
-#pragma unroll
-    for (int h = 0; h < GT; ++h) if (lane == 0) { sm_m[warp][h] = m[h]; sm_l[warp][h] = l[h]; }
+    if ((lane & ((WD_KEYS << SH) - 1)) == 0) { sm_m[warp][lane / (WD_KEYS << SH)] = m_l; sm_l[warp][lane / (WD_KEYS << SH)] = l_l; }
     const int unit = (r * L.G + kvh) * nhb + (blockIdx.x % nhb);
     float* my = R.attn_scratch + ((size_t)unit * R.splits + sp) * GT * (32 * EPL + 4);
 #pragma unroll
@@ -391,8 +409,13 @@ B2_API long long b2_window_attn_scratch(int H, int G, int dp, int rows, int spli
 B2_API int b2_window_attn_units(int H, int G, int rows) { return rows * G * ((H / G + WD_GT - 1) / WD_GT); }
 
 template <typename T, int EPL>
-static int launch_wd(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+static int launch_wd(const MixLayer* l, const MixRun* run, cudaStream_t s) {
     const int Gq = l->H / l->G;
+    // cache slices beyond what is resident at once would only add a second wave
+    MixRun one = *run;
+    const int units = l->G * ((Gq + WD_GT - 1) / WD_GT) * run->n_rows, slots = 148 * (Gq > 4 || EPL > 4 ? 1 : 2);
+    if (units * one.splits > slots) one.splits = units >= slots ? 1 : slots / units;
+    const MixRun* r = &one;
     // (a smaller head block keeps fewer registers; scratch is laid out for at most WD_GT heads per block)
     if (Gq <= 1) return launch_pdl(window_decode_kernel<T, EPL, 1>, dim3(l->G, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);
     if (Gq <= 2) return launch_pdl(window_decode_kernel<T, EPL, 2>, dim3(l->G, r->n_rows, r->splits), dim3(WD_THREADS), 0, s, *l, *r);

@@ -275,6 +275,7 @@ class Mix:
 SHAPES = [dict(), dict(H=12, G=1, d=32, rot=32, heads=5, P=33, N=17, groups=1, ngroups=5, taps=2),
           dict(H=3, G=3, d=100, rot=64, heads=2, P=72, N=130, groups=2, ngroups=1, taps=5),
           dict(H=8, G=2, d=64, rot=64, heads=8, P=64, N=128, groups=1, ngroups=2, taps=4),
+          dict(H=10, G=2, d=128, rot=96, heads=6, P=24, N=48, groups=3, ngroups=2, taps=3),
           dict(H=2, G=1, d=256, rot=128, heads=1, P=128, N=256, groups=1, ngroups=1, taps=1)]
 
 
