@@ -1,5 +1,6 @@
 """Shared test helpers: spawn gloo ranks on CPU, cosine similarity."""
 import os
+import pickle
 import socket
 import traceback
 
@@ -20,7 +21,9 @@ def _entry(rank, world, port, fn, args, q):
     torch.set_num_threads(1)
     try:
         dist.init_process_group("gloo", rank=rank, world_size=world)
-        q.put((rank, "ok", fn(rank, world, *args)))
+        # (pickled here: tensors sent as such are shared through a socket of this process, which may have ended
+        # by the time the parent opens it)
+        q.put((rank, "ok", pickle.dumps(fn(rank, world, *args))))
     except Exception:
         q.put((rank, "err", traceback.format_exc()))
     finally:
@@ -42,7 +45,7 @@ def run_gloo(fn, world: int, *args, timeout: float = 120.0):
             rank, status, val = q.get(timeout=timeout)
             if status != "ok":
                 raise RuntimeError(f"rank {rank} failed:\n{val}")
-            out[rank] = val
+            out[rank] = pickle.loads(val)
     finally:
         for p in procs:
             p.join(timeout=10)
