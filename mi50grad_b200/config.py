@@ -274,22 +274,38 @@ def memory_budget(config: QwenConfig, max_seq_len: int = 2048, num_gpus: int = 1
 
 
 # ---------------------------------------------------------------------------
-# Decoders whose layers are described one by one: a parallel mixer (windowed
-# attention beside a state-space recurrence) and a dense feed-forward, each with
-# a norm on its output only.
+# Decoders whose layers are described one by one: mixers made of windowed
+# attention and / or a linear recurrence, and a dense feed-forward.
 # ---------------------------------------------------------------------------
 
 @dataclass(frozen=True)
 class WindowAttentionSpec:
-    """Sliding-window attention whose values are the keys as projected; Q and K
-    are normalised over the whole projection."""
+    """Sliding-window attention."""
     heads: int
     kv_heads: int
     dim: int
-    rot_dims: int
+    rot_dims: int                     # 0: no rotation
     rot_base: float
     scale: float
     window: int                       # 0: unlimited
+    vdim: int = 0                     # size of a value head; 0: the values are the keys as projected
+    head_norm: bool = False           # Q and K normalised per head (one weight for all heads) or over the whole projection
+    keep_first: int = 0               # first tokens that stay visible beyond the window
+    softcap: float = 0.0              # scores become softcap * tanh(score / softcap); 0: none
+    sink: bool = False                # a learned number per head joins the soft-max's denominator
+
+    @property
+    def vd(self) -> int:
+        return self.vdim or self.dim
+
+    def check(self, where: str):
+        if (self.heads < 1 or self.kv_heads < 1 or self.heads % self.kv_heads or self.rot_dims % 2 or self.rot_dims > self.dim
+                or not 1 <= self.dim <= 256 or not 1 <= self.vd <= 256 or self.window < 0 or self.keep_first < 0):
+            raise ValueError(f"{where}: unsupported attention sizes {self}")
+
+    def cache_bytes_per_token(self, elem: int) -> int:
+        """A K and a V row (head rows padded to 8 elements)."""
+        return self.kv_heads * (-(-self.dim // 8) * 8 + -(-self.vd // 8) * 8) * elem
 
 
 @dataclass(frozen=True)
@@ -310,6 +326,40 @@ class SSDSpec:
     @property
     def conv_channels(self) -> int:
         return self.inner + 2 * self.groups * self.state
+
+    def check(self, where: str):
+        if self.heads % self.groups or self.inner % self.norm_groups or not 1 <= self.state <= 256 or self.conv < 1:
+            raise ValueError(f"{where}: unsupported recurrence sizes {self}")
+
+
+@dataclass(frozen=True)
+class LightningSpec:
+    """Linear attention S <- decay_h S + k v^T, o = S^T q with a constant decay per head; every head has its
+    own q and k (of size `state`) and v (of size `vdim`)."""
+    heads: int
+    state: int
+    vdim: int
+    decay: tuple
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    # no convolution in front of it
+    conv, conv_channels = 1, 0
+
+    def check(self, where: str):
+        if self.heads < 1 or self.vdim < 1 or not 1 <= self.state <= 256 or len(self.decay) != self.heads \
+                or any(not 0.0 <= x <= 1.0 for x in self.decay):
+            raise ValueError(f"{where}: unsupported recurrence sizes {self}")
+
+
+def _cache_bytes(mixers, max_seq_len: int, batch: int, elem: int) -> int:
+    return sum(batch * max_seq_len * a.cache_bytes_per_token(elem) for a, _ in mixers if a is not None)
+
+
+def _state_bytes(mixers, batch: int, elem: int) -> int:
+    return sum(batch * (s.heads * s.state * s.vdim * 4 + (s.conv - 1) * s.conv_channels * elem) for _, s in mixers if s is not None)
 
 
 @dataclass(frozen=True)
@@ -332,11 +382,8 @@ class DegedraConfig:
 
     def __post_init__(self):
         for i, l in enumerate(self.layers):
-            a, s = l.attention, l.ssd
-            if a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim or a.dim > 256:
-                raise ValueError(f"layer {i}: unsupported attention sizes {a}")
-            if s.heads % s.groups or s.inner % s.norm_groups or s.state > 256 or s.conv < 1:
-                raise ValueError(f"layer {i}: unsupported recurrence sizes {s}")
+            l.attention.check(f"layer {i}")
+            l.ssd.check(f"layer {i}")
             self.weight_layer(i)
 
     @property
@@ -353,14 +400,19 @@ class DegedraConfig:
                 raise ValueError("weights_of does not lead to a layer with tensors")
         return i
 
+    def run_order(self) -> List[int]:
+        """Layer of every run of a layer in a step."""
+        return list(range(len(self.layers)))
+
+    def run_mixers(self) -> list:
+        """(attention or None, recurrence or None) of every run: what it keeps in the cache and the state."""
+        return [(l.attention, l.ssd) for l in self.layers]
+
     def cache_bytes(self, max_seq_len: int, batch: int = 1, elem: int = 2) -> int:
-        """K and V rows of every layer (head rows padded to 8 elements)."""
-        return sum(2 * batch * max_seq_len * l.attention.kv_heads * (-(-l.attention.dim // 8) * 8) * elem
-                   for l in self.layers)
+        return _cache_bytes(self.run_mixers(), max_seq_len, batch, elem)
 
     def state_bytes(self, batch: int = 1, elem: int = 2) -> int:
-        return sum(batch * (l.ssd.heads * l.ssd.state * l.ssd.vdim * 4 + (l.ssd.conv - 1) * l.ssd.conv_channels * elem)
-                   for l in self.layers)
+        return _state_bytes(self.run_mixers(), batch, elem)
 
 
 def tiny_degedra_config() -> DegedraConfig:
@@ -412,6 +464,128 @@ def degedra_config_to_dict(cfg: DegedraConfig) -> dict:
            "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
     if cfg.logit_softcap:
         out["logit_softcap"] = cfg.logit_softcap
+    return out
+
+
+# Vekerax: pre-norm decoder over several residual streams, each layer with one mixer (attention or lightning
+# attention), some of the layers run several times with the same weights.
+
+@dataclass(frozen=True)
+class StreamLayerSpec:
+    """One mixer (a `WindowAttentionSpec` or a `LightningSpec`) and a feed-forward."""
+    mixer: object
+    ff: int = 0                       # 0: no feed-forward
+    act: str = "relu"                 # of the feed-forward's gate
+
+    @property
+    def attention(self) -> Optional[WindowAttentionSpec]:
+        return self.mixer if isinstance(self.mixer, WindowAttentionSpec) else None
+
+    @property
+    def recurrence(self) -> Optional[LightningSpec]:
+        return self.mixer if isinstance(self.mixer, LightningSpec) else None
+
+
+MAX_STREAMS = 16
+
+
+@dataclass
+class VekeraxConfig:
+    hidden_size: int
+    vocab_size: int
+    rms_norm_eps: float
+    layers: List[StreamLayerSpec]
+    embedding_scale: float = 1.0
+    residual_mult: float = 1.0
+    streams: int = 0                  # residual streams joined by hyper-connections; 0: one stream, plain residual sums
+    loop: Optional[tuple] = None      # (start, stop, times): layers start .. stop-1 run `times` times in a row
+
+    def __post_init__(self):
+        for i, l in enumerate(self.layers):
+            l.mixer.check(f"layer {i}")
+        if not 0 <= self.streams <= MAX_STREAMS:
+            raise ValueError(f"at most {MAX_STREAMS} residual streams")
+        if self.loop is not None:
+            a, b, n = self.loop
+            if not 0 <= a <= b <= len(self.layers) or n < 0:
+                raise ValueError(f"the loop {self.loop} does not fit {len(self.layers)} layers")
+
+    @property
+    def num_hidden_layers(self) -> int:
+        """Layers with weights (a looped one counts once)."""
+        return len(self.layers)
+
+    def run_order(self) -> List[int]:
+        """Layer of every run of a layer in a step."""
+        n = len(self.layers)
+        if self.loop is None:
+            return list(range(n))
+        a, b, times = self.loop
+        return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+
+    def run_mixers(self) -> list:
+        """(attention or None, recurrence or None) of every run: each has a cache or state of its own."""
+        return [(self.layers[i].attention, self.layers[i].recurrence) for i in self.run_order()]
+
+    def cache_bytes(self, max_seq_len: int, batch: int = 1, elem: int = 2) -> int:
+        return _cache_bytes(self.run_mixers(), max_seq_len, batch, elem)
+
+    def state_bytes(self, batch: int = 1, elem: int = 2) -> int:
+        return _state_bytes(self.run_mixers(), batch, elem)
+
+
+def tiny_vekerax_config() -> VekeraxConfig:
+    """Three small layers, two of them run three times, three streams (smoke runs, examples)."""
+    a = WindowAttentionSpec(6, 2, 48, 0, 0.0, 48 ** -0.5, 40, vdim=32, head_norm=True, keep_first=3, softcap=20.0, sink=True)
+    s = LightningSpec(4, 24, 40, (0.5, 0.9, 0.99, 1.0))
+    return VekeraxConfig(256, 1000, 1e-6, [StreamLayerSpec(a, 320), StreamLayerSpec(s, 320), StreamLayerSpec(a)], 2.0, 0.6, 3, (1, 3, 3))
+
+
+def vekerax_config_from_dict(c: dict) -> VekeraxConfig:
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        if e.get("type") == "attention":
+            mask = m.get("mask") or {}
+            mixer = WindowAttentionSpec(m["heads"], m["kv_heads"], m["dim"], 0, 0.0, float(m["scale"]), int(mask.get("size") or 0),
+                                        vdim=m["vdim"], head_norm=True, keep_first=int(mask.get("keep_first") or 0),
+                                        softcap=float(m.get("softcap") or 0.0), sink=True)
+        elif e.get("type") == "lightning":
+            mixer = LightningSpec(m["heads"], m["dim"], m["vdim"], tuple(float(x) for x in m["decay"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        layers.append(StreamLayerSpec(mixer, 0 if mlp is None else mlp["ff"]))
+    loop = c.get("loop")
+    return VekeraxConfig(hidden_size=c["width"], vocab_size=c["vocab"], rms_norm_eps=float(c["norm"]["eps"]), layers=layers,
+                         embedding_scale=float((c.get("embedding") or {}).get("scale", 1.0)),
+                         residual_mult=float(c.get("residual_mult", 1.0)), streams=int(c.get("streams") or 0),
+                         loop=None if not loop else (loop["start"], loop["stop"], loop["times"]))
+
+
+def vekerax_config_to_dict(cfg: VekeraxConfig) -> dict:
+    """The config.json form that `vekerax_config_from_dict` reads."""
+    layers = []
+    for l in cfg.layers:
+        if l.attention is not None:
+            a = l.attention
+            e = {"type": "attention", "mixer": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vd, "scale": a.scale}}
+            if a.softcap:
+                e["mixer"]["softcap"] = a.softcap
+            if a.window:
+                e["mixer"]["mask"] = {"size": a.window, "keep_first": a.keep_first}
+        else:
+            r = l.recurrence
+            e = {"type": "lightning", "mixer": {"heads": r.heads, "dim": r.state, "vdim": r.vdim, "decay": list(r.decay)}}
+        e["mlp"] = {"kind": "dense", "ff": l.ff} if l.ff else None
+        layers.append(e)
+    out = {"architecture": "Vekerax", "width": cfg.hidden_size, "vocab": cfg.vocab_size, "norm": {"eps": cfg.rms_norm_eps},
+           "embedding": {"scale": cfg.embedding_scale}, "residual_mult": cfg.residual_mult, "layers": layers}
+    if cfg.streams:
+        out["streams"] = cfg.streams
+    if cfg.loop is not None:
+        out["loop"] = dict(zip(("start", "stop", "times"), cfg.loop))
     return out
 
 

@@ -1,15 +1,18 @@
-// Sliding-window attention of a parallel mixer, and the preparation pass in front of both of its branches.
+// Sliding-window attention, and the preparation pass in front of a mixer.
 //
-//   mix_prepare       RMSNorm of Q and of K over the WHOLE projection (all heads at once), rotation of the
-//                     first `rot` dimensions of every head in (i, i + rot/2) pairs, K and the values (K as
-//                     projected) into the cache, causal convolution + SiLU of the recurrence's inputs, its
-//                     step sizes.
+//   mix_prepare       parallel mixer: RMSNorm of Q and of K over the WHOLE projection (all heads at once), rotation
+//                     of the first `rot` dimensions of every head in (i, i + rot/2) pairs, K and the values into the
+//                     cache, causal convolution + SiLU of the recurrence's inputs, its step sizes.
+//   head_prepare      attention alone: RMSNorm of every Q and K head with one weight for all heads, optional
+//                     rotation, K and the values into the cache.
 //   window decode     split-KV flash decoding, any head size up to 256, bf16 or fp32 cache.
 //   window rows       many query rows of one sequence: 64-row tiles on bf16 tensor cores (mma.sync) that
 //                     walk only the key blocks their windows reach.
 //
-// Visibility: the row at position p sees slots max(0, p - window + 1) .. p of its sequence (slot = position:
-// rows of a sequence are consecutive tokens, no draft trees).
+// Visibility: the row at position p sees slots max(0, p - window + 1) .. p of its sequence and its first
+// keep_first slots (slot = position: rows of a sequence are consecutive tokens, no draft trees).  Scores may be
+// capped (softcap * tanh(score / softcap)), and a learned sink per head may join the soft-max's denominator: it
+// is neither scaled nor capped and has no value.
 #include "mixers.cuh"
 
 // ---------------------------------------------------------------------------
@@ -34,7 +37,7 @@ __device__ __forceinline__ void mp_heads(const MixLayer& L, const MixRun& R, int
     const float* nw = is_q ? L.q_norm : L.k_norm;
     const size_t slot = ((size_t)rm.seq * L.max_seq + rm.slot) * L.G * L.dp;
     T* dst = is_q ? (T*)R.qbuf + (size_t)r * L.H * L.dp : (T*)L.kcache + slot;
-    T* vdst = (T*)L.vcache + slot;
+    T* vdst = (T*)L.vcache + slot;                         // (values = keys as projected: vp == dp)
     constexpr int V = 16 / sizeof(T);
     const bool vec = ((off | R.ld_proj | n) & (V - 1)) == 0;
     pdl_wait();
@@ -166,7 +169,102 @@ __global__ void __launch_bounds__(MP_THREADS) mix_prepare_kernel(const MixLayer 
     mp_conv<T>(L, R, b % col_blocks, r0, min(conv_rows, R.n_rows - r0));
 }
 
+// ---------------------------------------------------------------------------
+// head_prepare: one warp per (row, query head | key head | value head)
+// ---------------------------------------------------------------------------
+template <typename T, int EPL>
+__global__ void __launch_bounds__(256) head_prepare_kernel(const MixLayer L, const MixRun R) {
+    __shared__ float sv[8][32 * EPL];
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per = L.H + L.G + (L.off_v >= 0 ? L.G : 0), unit = blockIdx.x * 8 + warp;
+    if (unit >= R.n_rows * per) return;
+    const int r = unit / per, j = unit % per;
+    const RowMeta rm = R.rows[r];
+    const bool is_q = j < L.H, is_v = j >= L.H + L.G;
+    const int hd = is_q ? j : (is_v ? j - L.H - L.G : j - L.H), n = is_v ? L.dv : L.d, np = is_v ? L.vp : L.dp;
+    const int off = (is_q ? L.off_q : (is_v ? L.off_v : L.off_k)) + hd * n, c0 = lane * EPL;
+    const T* src = (const T*)R.proj + (size_t)r * R.ld_proj + off + c0;
+    const size_t slot = ((size_t)rm.seq * L.max_seq + rm.slot) * L.G + hd;
+    T* dst = is_q ? (T*)R.qbuf + ((size_t)r * L.H + hd) * L.dp : (is_v ? (T*)L.vcache + slot * L.vp : (T*)L.kcache + slot * L.dp);
+    const float* nw = is_q ? L.q_norm : L.k_norm;
+    const bool vec = ((off | n | R.ld_proj) & (EPL - 1)) == 0;
+    float w[EPL], v[EPL], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) w[e] = (!is_v && c0 + e < n) ? nw[c0 + e] : 0.f;
+    pdl_wait();
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) v[e] = 0.f;
+    if (vec && c0 < n) {
+        T raw[EPL];
+        if constexpr (EPL * sizeof(T) == 4) *(uint32_t*)raw = *(const uint32_t*)src;
+        else if constexpr (EPL * sizeof(T) == 8) *(uint2*)raw = *(const uint2*)src;
+        else
+#pragma unroll
+            for (int i = 0; i < (int)(EPL * sizeof(T) / 16); ++i) ((uint4*)raw)[i] = ((const uint4*)src)[i];
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) v[e] = ld_f(raw + e);
+    } else
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) if (c0 + e < n) v[e] = ld_f(src + e);
+    auto put = [&](T* d, int len, const float (&o)[EPL]) {          // (len is a multiple of 8)
+        if (c0 >= len) return;
+        T raw[EPL];
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) raw[e] = to_t<T>(o[e]);
+        if constexpr (EPL * sizeof(T) == 4) *(uint32_t*)(d + c0) = *(const uint32_t*)raw;
+        else if constexpr (EPL * sizeof(T) == 8) *(uint2*)(d + c0) = *(const uint2*)raw;
+        else
+#pragma unroll
+            for (int i = 0; i < (int)(EPL * sizeof(T) / 16); ++i) ((uint4*)(d + c0))[i] = ((const uint4*)raw)[i];
+    };
+    if (is_v) { put(dst, np, v); return; }
+    if (!is_q && L.off_v < 0) put((T*)L.vcache + slot * L.vp, L.vp, v);
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) ss += v[e] * v[e];
+    const float inv = rsqrtf(warp_sum(ss) / (float)n + L.eps);
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) v[e] *= inv * w[e];
+    if (L.rot > 0) {
+        const int half = L.rot >> 1;
+        const float* ct = L.cos_tab + (size_t)rm.pos * half;
+        const float* st = L.sin_tab + (size_t)rm.pos * half;
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) sv[warp][c0 + e] = v[e];
+        __syncwarp();
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) {
+            const int i = c0 + e;
+            if (i >= L.rot) continue;
+            const bool first = i < half;
+            const int a = first ? i : i - half;
+            const float other = sv[warp][first ? i + half : a];
+            v[e] = first ? v[e] * ct[a] - other * st[a] : v[e] * ct[a] + other * st[a];
+        }
+    }
+    put(dst, np, v);
+}
+template <typename T>
+static int launch_hp(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    const int per = l->H + l->G + (l->off_v >= 0 ? l->G : 0), m = l->dp > l->vp ? l->dp : l->vp;
+    const dim3 grid((r->n_rows * per + 7) / 8), block(256);
+    if (m <= 64) return launch_pdl(head_prepare_kernel<T, 2>, grid, block, 0, s, *l, *r);
+    if (m <= 128) return launch_pdl(head_prepare_kernel<T, 4>, grid, block, 0, s, *l, *r);
+    return launch_pdl(head_prepare_kernel<T, 8>, grid, block, 0, s, *l, *r);
+}
+
+static bool attn_valid(const MixLayer* l) {
+    return l->H >= 1 && l->G >= 1 && l->H % l->G == 0 && l->d >= 1 && l->dp >= l->d && l->dp <= 256 && !(l->dp & 7) && l->dv >= 1 &&
+           l->vp >= l->dv && l->vp <= 256 && !(l->vp & 7) && l->rot <= l->d && !(l->rot & 1) && l->keep_first >= 0;
+}
+B2_API int b2_head_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (!attn_valid(l) || !l->head_norm || !l->q_norm || !l->k_norm || (l->off_v < 0 && l->dv != l->d) || (l->rot > 0 && !l->cos_tab))
+        return cudaErrorInvalidValue;
+    return r->dt == DT_BF16 ? launch_hp<bf16>(l, r, s) : launch_hp<float>(l, r, s);
+}
+
 B2_API int b2_mix_prepare(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    if (!attn_valid(l) || l->head_norm || l->off_v >= 0 || l->dv != l->d) return cudaErrorInvalidValue;
     if (l->H < 1 || l->G < 1 || l->H % l->G || l->d > 256 || l->dp < l->d || (l->dp & 7) || l->rot > l->d || (l->rot & 1) ||
         l->taps < 1 || l->groups < 1 || l->heads % l->groups)
         return cudaErrorInvalidValue;
@@ -231,17 +329,18 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
     const RowMeta rm = R.rows[r];
     const int k1 = rm.pos + 1;                                               // keys [k0, k1)
     const int k0 = L.window > 0 ? max(0, k1 - L.window) : 0;
-    const int total = k1 - k0;
+    // the keys a row sees, in order: kf kept first ones, then its window
+    const int kf = min(L.keep_first, k0), total = kf + k1 - k0, jump = k0 - kf;
     const int nsplit = max(1, min(R.splits, (total + WD_MIN_SPLIT - 1) / WD_MIN_SPLIT));
     if (sp >= nsplit) return;
     const int per = (total + nsplit - 1) / nsplit;
-    const int a0 = k0 + sp * per, a1 = min(k1, a0 + per);
+    const int a0 = sp * per, a1 = min(total, a0 + per);
     __shared__ float sm_m[WD_WARPS][GT], sm_l[WD_WARPS][GT], sm_f[WD_MAX_SPLITS][GT], sm_li[GT];
     __shared__ float sm_acc[WD_WARPS][32 * EPL];
     __shared__ int s_last;
     pdl_wait();
-    const bool in = lane * EPL < L.dp;                       // dp is a multiple of EPL (<= 8): lanes are in or out as a whole
     const int col = lane * EPL;
+    const bool in = col < L.dp, in_v = col < L.vp;           // multiples of EPL (<= 8): lanes are in or out as a whole
     // Scores of WD_KEYS keys x GT heads are summed over the lanes by recursive halving: every step a lane hands
     // half of its values to its partner and keeps the other half, so afterwards each lane holds ONE finished
     // score (the value with index lane >> SH) and the soft-max costs one exponential per lane.  The running
@@ -256,17 +355,17 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
 #pragma unroll
         for (int e = 0; e < EPL; ++e) { q[h][e] = wr_get(qv, e) * L.attn_scale; acc[h][e] = 0.f; }
     }
-    const size_t base = ((size_t)rm.seq * L.max_seq * L.G + kvh) * L.dp + col, stride = (size_t)L.G * L.dp;
-    const T* kc = (const T*)L.kcache + base;
-    const T* vc = (const T*)L.vcache + base;
+    const size_t base = (size_t)rm.seq * L.max_seq * L.G + kvh, stride = (size_t)L.G * L.dp, vstride = (size_t)L.G * L.vp;
+    const T* kc = (const T*)L.kcache + base * L.dp + col;
+    const T* vc = (const T*)L.vcache + base * L.vp + col;
     WRaw<T, EPL> kn[WD_KEYS], vn[WD_KEYS];
     auto fetch = [&](int s) {
 #pragma unroll
         for (int i = 0; i < WD_KEYS; ++i) {
-            const int key = s + i * WD_WARPS + warp;
-            const bool ok = in && key < a1;
-            wr_load(kn[i], kc + (size_t)key * stride, ok);
-            wr_load(vn[i], vc + (size_t)key * stride, ok);
+            const int idx = s + i * WD_WARPS + warp, key = idx < kf ? idx : idx + jump;
+            const bool ok = idx < a1;
+            wr_load(kn[i], kc + (size_t)key * stride, in && ok);
+            wr_load(vn[i], vc + (size_t)key * vstride, in_v && ok);
         }
     };
     if (a0 < a1) fetch(a0);
@@ -298,6 +397,7 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
         }
 #pragma unroll
         for (int o = 16 / NV; o > 0; o >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], o);
+        if (L.softcap > 0.f) d[0] = L.softcap * tanhf(d[0] / L.softcap);
         const float sc = s + mykey * WD_WARPS + warp < a1 ? d[0] : -INFINITY;
         float mn = sc;
 #pragma unroll
@@ -339,14 +439,17 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
         float mm = -INFINITY;
 #pragma unroll
         for (int w = 0; w < WD_WARPS; ++w) mm = fmaxf(mm, sm_m[w][h]);
-        float ll = 0.f, f[WD_WARPS];
+        const int head = kvh * Gq + hb + h;
+        const bool sink = L.sink && nsplit == 1;             // (slices: the merge below counts it)
+        if (sink) mm = fmaxf(mm, L.sink[head]);
+        float ll = sink ? expf(L.sink[head] - mm) : 0.f, f[WD_WARPS];
 #pragma unroll
         for (int w = 0; w < WD_WARPS; ++w) { f[w] = sm_m[w][h] == -INFINITY ? 0.f : expf(sm_m[w][h] - mm); ll += sm_l[w][h] * f[w]; }
-        for (int c = tid; c < L.d; c += WD_THREADS) {
+        for (int c = tid; c < L.dv; c += WD_THREADS) {
             float a = 0.f;
 #pragma unroll
             for (int w = 0; w < WD_WARPS; ++w) a += sm_acc[w][c] * f[w];
-            if (nsplit == 1) ((T*)R.out)[(size_t)r * R.ldo + (kvh * Gq + hb + h) * L.d + c] = to_t<T>(a / ll * L.left_scale);
+            if (nsplit == 1) ((T*)R.out)[(size_t)r * R.ldo + head * L.dv + c] = to_t<T>(a / ll * L.left_scale);
             else {
                 my[h * (32 * EPL + 4) + c] = a;
                 if (c == 0) { my[h * (32 * EPL + 4) + 32 * EPL] = mm; my[h * (32 * EPL + 4) + 32 * EPL + 1] = ll; }
@@ -377,6 +480,7 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
         }
 #pragma unroll
         for (int x = 0; x < WD_MAX_SPLITS; ++x) mm = fmaxf(mm, mv[x]);
+        if (L.sink) { const float sk = L.sink[kvh * Gq + hb + tid]; mm = fmaxf(mm, sk); ll = expf(sk - mm); }
 #pragma unroll
         for (int x = 0; x < WD_MAX_SPLITS; ++x) {
             const float f = mv[x] == -INFINITY ? 0.f : expf(mv[x] - mm);
@@ -386,8 +490,8 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
         sm_li[tid] = 1.f / ll;
     }
     __syncthreads();
-    for (int i = tid; i < nh * L.d; i += WD_THREADS) {
-        const int h = i / L.d, c = i % L.d;
+    for (int i = tid; i < nh * L.dv; i += WD_THREADS) {
+        const int h = i / L.dv, c = i % L.dv;
         float a = 0.f;
         for (int x0 = 0; x0 < nsplit; x0 += 8) {
             float v[8];
@@ -397,11 +501,11 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(const MixLaye
 #pragma unroll
             for (int u = 0; u < 8; ++u) if (x0 + u < nsplit) a = fmaf(v[u], sm_f[x0 + u][h], a);
         }
-        ((T*)R.out)[(size_t)r * R.ldo + (kvh * Gq + hb + h) * L.d + c] = to_t<T>(a * sm_li[h] * L.left_scale);
+        ((T*)R.out)[(size_t)r * R.ldo + (kvh * Gq + hb + h) * L.dv + c] = to_t<T>(a * sm_li[h] * L.left_scale);
     }
 }
 
-// floats of scratch for `rows` rows (attn_counters: rows * G * ceil(H / G / WD_GT) ints)
+// floats of scratch for `rows` rows, dp: the larger of MixLayer's dp and vp (attn_counters: rows * G * ceil(H / G / WD_GT) ints)
 B2_API long long b2_window_attn_scratch(int H, int G, int dp, int rows, int splits) {
     const int nhb = (H / G + WD_GT - 1) / WD_GT, epl = dp <= 64 ? 2 : dp <= 128 ? 4 : 8;
     return (long long)rows * G * nhb * splits * WD_GT * (32 * epl + 4);
@@ -425,12 +529,13 @@ static int launch_wd(const MixLayer* l, const MixRun* run, cudaStream_t s) {
 }
 template <typename T>
 static int launch_wd_t(const MixLayer* l, const MixRun* r, cudaStream_t s) {
-    if (l->dp <= 64) return launch_wd<T, 2>(l, r, s);
-    if (l->dp <= 128) return launch_wd<T, 4>(l, r, s);
+    const int m = l->dp > l->vp ? l->dp : l->vp;
+    if (m <= 64) return launch_wd<T, 2>(l, r, s);
+    if (m <= 128) return launch_wd<T, 4>(l, r, s);
     return launch_wd<T, 8>(l, r, s);
 }
 B2_API int b2_window_attn_decode(const MixLayer* l, const MixRun* r, cudaStream_t s) {
-    if (l->dp > 256 || (l->dp & 7) || l->H % l->G || r->splits < 1 || r->splits > WD_MAX_SPLITS) return cudaErrorInvalidValue;
+    if (!attn_valid(l) || r->splits < 1 || r->splits > WD_MAX_SPLITS) return cudaErrorInvalidValue;
     return r->dt == DT_BF16 ? launch_wd_t<bf16>(l, r, s) : launch_wd_t<float>(l, r, s);
 }
 
@@ -459,7 +564,20 @@ __device__ __forceinline__ uint32_t wr_pack(float x, float y) {
     return *(const uint32_t*)&h;
 }
 
-template <int DP>
+// v = t[0] + .. + t[TERMS - 1] with bf16 terms of two values each
+template <int TERMS>
+__device__ __forceinline__ void wr_split(float a, float b, uint32_t (&t)[TERMS]) {
+#pragma unroll
+    for (int i = 0; i < TERMS; ++i) {
+        t[i] = wr_pack(a, b);
+        if (i + 1 < TERMS) { a -= __uint_as_float(t[i] << 16); b -= __uint_as_float(t[i] & 0xffff0000u); }
+    }
+}
+// cap * tanh(x / cap) = cap - 2 cap / (1 + exp(2 x / cap)); e = 2 log2(e) / cap
+__device__ __forceinline__ float wr_cap(float x, float cap, float e) { return cap - __fdividef(2.f * cap, 1.f + exp2f(x * e)); }
+
+// TERMS: bf16 terms of a soft-max weight in the product with V (1: the weight rounded to bf16, 3: all of its 24 bits)
+template <int DP, int TERMS>
 __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, const MixRun R) {
     constexpr int LD = DP + WR_PAD, NT_O = DP / 8, PPR = DP / 8;
     extern __shared__ __align__(16) unsigned char wrs[];
@@ -474,7 +592,9 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
     const int p0 = rm.pos;                       // positions of the tile: p0 .. p0 + nrows - 1
     const int k_lo = L.window > 0 ? max(0, p0 - L.window + 1) : 0, k_hi = p0 + nrows;
     const int b0 = k_lo / WR_KEYS, b1 = (k_hi + WR_KEYS - 1) / WR_KEYS;
-    const size_t kv_base = ((size_t)rm.seq * L.max_seq * L.G + kvh) * L.dp, kv_stride = (size_t)L.G * L.dp;
+    // blocks walked: those of the kept first keys in front of b0, then b0 .. b1 - 1
+    const int kept = min(b0, (L.keep_first + WR_KEYS - 1) / WR_KEYS), n_blk = kept + b1 - b0;
+    const size_t kv_base = (size_t)rm.seq * L.max_seq * L.G + kvh;
     pdl_wait();
     for (int i = tid; i < WR_ROWS * PPR; i += 128) {
         const int pc = i % PPR, r = i / PPR;
@@ -487,16 +607,13 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
             const int pc = i % PPR, r = i / PPR, slot = blk * WR_KEYS + r;
             bf16* kd = Kb + (buf * WR_KEYS + r) * LD + pc * 8;
             bf16* vd = Vb + (buf * WR_KEYS + r) * LD + pc * 8;
-            if (slot < k_hi && pc * 8 < L.dp) {
-                cp_async16(kd, (const bf16*)L.kcache + kv_base + (size_t)slot * kv_stride + pc * 8);
-                cp_async16(vd, (const bf16*)L.vcache + kv_base + (size_t)slot * kv_stride + pc * 8);
-            } else {
-                *(uint4*)kd = make_uint4(0u, 0u, 0u, 0u);
-                *(uint4*)vd = make_uint4(0u, 0u, 0u, 0u);
-            }
+            if (slot < k_hi && pc * 8 < L.dp) cp_async16(kd, (const bf16*)L.kcache + (kv_base + (size_t)slot * L.G) * L.dp + pc * 8);
+            else *(uint4*)kd = make_uint4(0u, 0u, 0u, 0u);
+            if (slot < k_hi && pc * 8 < L.vp) cp_async16(vd, (const bf16*)L.vcache + (kv_base + (size_t)slot * L.G) * L.vp + pc * 8);
+            else *(uint4*)vd = make_uint4(0u, 0u, 0u, 0u);
         }
     };
-    stage(b0, 0);
+    stage(kept > 0 ? 0 : b0, 0);
     cp_async_commit();
     float o[NT_O][4];
 #pragma unroll
@@ -505,18 +622,21 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
     const bf16* qw = Qs + warp * 16 * LD;
     const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
     const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;
-    const float sc = L.attn_scale * 1.44269504f;             // scores in the log2 domain
+    constexpr float LOG2E = 1.44269504f;                     // scores end up in the log2 domain
+    const float cap = L.softcap, cap_e = cap > 0.f ? 2.f * LOG2E / cap : 0.f;
+    const float sc = cap > 0.f ? L.attn_scale : L.attn_scale * LOG2E;
     const int q_lo = p0 + warp * 16 + g, q_hi = q_lo + 8;    // positions of this thread's two rows
     const int w_lo = L.window > 0 ? q_lo - L.window : -1, w_hi = L.window > 0 ? q_hi - L.window : -1;     // last invisible slots
     const int wp0 = p0 + warp * 16;                          // the warp's positions: wp0 .. wp0 + 15
-    for (int blk = b0; blk < b1; ++blk) {
-        const int buf = (blk - b0) & 1, s_base = blk * WR_KEYS;
+    for (int it = 0; it < n_blk; ++it) {
+        auto block_of = [&](int i) { return i < kept ? i : i - kept + b0; };
+        const int buf = it & 1, s_base = block_of(it) * WR_KEYS;
         cp_async_wait<0>();
         __syncthreads();
-        if (blk + 1 < b1) stage(blk + 1, buf ^ 1);
+        if (it + 1 < n_blk) stage(block_of(it + 1), buf ^ 1);
         cp_async_commit();
         // nothing of this block is visible to the warp's rows
-        if (s_base > wp0 + 15 || (L.window > 0 && s_base + WR_KEYS - 1 <= wp0 - L.window) || warp * 16 >= nrows) continue;
+        if (s_base > wp0 + 15 || (L.window > 0 && s_base + WR_KEYS - 1 <= wp0 - L.window && s_base >= L.keep_first) || warp * 16 >= nrows) continue;
         const bf16* Kt = Kb + buf * WR_KEYS * LD;
         const bf16* Vt = Vb + buf * WR_KEYS * LD;
         float s[WR_KEYS / 8][4];
@@ -535,15 +655,17 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
             }
         }
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
-        const bool whole = s_base + WR_KEYS - 1 <= wp0 && (L.window <= 0 || s_base > wp0 + 15 - L.window);
+        const bool whole = s_base + WR_KEYS - 1 <= wp0 && (L.window <= 0 || s_base > wp0 + 15 - L.window || s_base + WR_KEYS <= L.keep_first);
 #pragma unroll
         for (int n = 0; n < WR_KEYS / 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float v = s[n][e] * sc;
+                if (cap > 0.f) v = wr_cap(v, cap, cap_e) * LOG2E;
                 if (!whole) {
                     const int slot = s_base + 8 * n + 2 * t + (e & 1);
-                    const bool vis = e >= 2 ? (slot <= q_hi && slot > w_hi) : (slot <= q_lo && slot > w_lo);
+                    const bool vis = e >= 2 ? (slot <= q_hi && (slot > w_hi || slot < L.keep_first))
+                                            : (slot <= q_lo && (slot > w_lo || slot < L.keep_first));
                     if (!vis) v = -INFINITY;
                 }
                 s[n][e] = v;
@@ -556,62 +678,78 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
         const float c_lo = exp2f(m_lo - rf_lo), c_hi = exp2f(m_hi - rf_hi);
         m_lo = mn_lo; m_hi = mn_hi;
         float rs_lo = 0.f, rs_hi = 0.f;
-        uint32_t pa[WR_KEYS / 16][4];
 #pragma unroll
         for (int n = 0; n < WR_KEYS / 8; ++n) {
-            const float e0 = exp2f(s[n][0] - rf_lo), e1 = exp2f(s[n][1] - rf_lo);
-            const float e2 = exp2f(s[n][2] - rf_hi), e3 = exp2f(s[n][3] - rf_hi);
-            rs_lo += e0 + e1; rs_hi += e2 + e3;
-            pa[n >> 1][(n & 1) * 2 + 0] = wr_pack(e0, e1);
-            pa[n >> 1][(n & 1) * 2 + 1] = wr_pack(e2, e3);
+            s[n][0] = exp2f(s[n][0] - rf_lo); s[n][1] = exp2f(s[n][1] - rf_lo);
+            s[n][2] = exp2f(s[n][2] - rf_hi); s[n][3] = exp2f(s[n][3] - rf_hi);
+            rs_lo += s[n][0] + s[n][1]; rs_hi += s[n][2] + s[n][3];
         }
         l_lo = l_lo * c_lo + rs_lo; l_hi = l_hi * c_hi + rs_hi;
 #pragma unroll
         for (int n = 0; n < NT_O; ++n) { o[n][0] *= c_lo; o[n][1] *= c_lo; o[n][2] *= c_hi; o[n][3] *= c_hi; }
 #pragma unroll
-        for (int k16 = 0; k16 < WR_KEYS / 16; ++k16)
+        for (int k16 = 0; k16 < WR_KEYS / 16; ++k16) {
+            uint32_t t0[TERMS], t1[TERMS], t2[TERMS], t3[TERMS];
+            wr_split<TERMS>(s[2 * k16][0], s[2 * k16][1], t0);
+            wr_split<TERMS>(s[2 * k16][2], s[2 * k16][3], t1);
+            wr_split<TERMS>(s[2 * k16 + 1][0], s[2 * k16 + 1][1], t2);
+            wr_split<TERMS>(s[2 * k16 + 1][2], s[2 * k16 + 1][3], t3);
 #pragma unroll
             for (int np = 0; np < NT_O / 2; ++np) {
                 uint32_t b[4];
                 wr_ldsm4_t(b, Vt + (k16 * 16 + a_row) * LD + np * 16 + a_col);
-                wr_mma(o[2 * np], pa[k16], b[0], b[1]);
-                wr_mma(o[2 * np + 1], pa[k16], b[2], b[3]);
+#pragma unroll
+                for (int i = 0; i < TERMS; ++i) {
+                    const uint32_t pa[4] = {t0[i], t1[i], t2[i], t3[i]};
+                    wr_mma(o[2 * np], pa, b[0], b[1]);
+                    wr_mma(o[2 * np + 1], pa, b[2], b[3]);
+                }
             }
+        }
     }
     cp_async_wait<0>();
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+    if (L.sink) {
+        const float sk = L.sink[head] * LOG2E;
+        l_lo += exp2f(sk - m_lo); l_hi += exp2f(sk - m_hi);
+    }
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
         const int rr = warp * 16 + g + 8 * half;
         if (rr >= nrows) continue;
         const float f = L.left_scale / (half ? l_hi : l_lo);
-        bf16* dst = (bf16*)R.out + (size_t)(row0 + rr) * R.ldo + (size_t)head * L.d;
+        bf16* dst = (bf16*)R.out + (size_t)(row0 + rr) * R.ldo + (size_t)head * L.dv;
 #pragma unroll
         for (int n = 0; n < NT_O; ++n)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int c = 8 * n + 2 * t + e;
-                if (c < L.d) dst[c] = __float2bfloat16(o[n][2 * half + e] * f);
+                if (c < L.dv) dst[c] = __float2bfloat16(o[n][2 * half + e] * f);
             }
     }
 }
 
-template <int DP>
+template <int DP, int TERMS>
 static int launch_wr(const MixLayer* l, const MixRun* r, cudaStream_t s) {
     const size_t smem = (size_t)(WR_ROWS + 4 * WR_KEYS) * (DP + WR_PAD) * sizeof(bf16);
     static SmemOptIn opt;
-    if (int e = opt.ensure((const void*)window_rows_kernel<DP>, smem)) return e;
-    return launch_pdl(window_rows_kernel<DP>, dim3((r->n_rows + WR_ROWS - 1) / WR_ROWS, l->H), dim3(128), smem, s, *l, *r);
+    if (int e = opt.ensure((const void*)window_rows_kernel<DP, TERMS>, smem)) return e;
+    return launch_pdl(window_rows_kernel<DP, TERMS>, dim3((r->n_rows + WR_ROWS - 1) / WR_ROWS, l->H), dim3(128), smem, s, *l, *r);
+}
+template <int TERMS>
+static int launch_wr_t(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    const int m = l->dp > l->vp ? l->dp : l->vp;
+    if (m <= 32) return launch_wr<32, TERMS>(l, r, s);
+    if (m <= 64) return launch_wr<64, TERMS>(l, r, s);
+    if (m <= 96) return launch_wr<96, TERMS>(l, r, s);
+    if (m <= 128) return launch_wr<128, TERMS>(l, r, s);
+    return launch_wr<256, TERMS>(l, r, s);
 }
 // All rows belong to one sequence, bf16 only (b2_window_attn_decode takes everything else).
 B2_API int b2_window_attn_rows(const MixLayer* l, const MixRun* r, cudaStream_t s) {
-    if (r->dt != DT_BF16 || r->n_seqs != 1 || l->dp > 256 || (l->dp & 7) || l->H % l->G) return cudaErrorInvalidValue;
-    if (l->dp <= 32) return launch_wr<32>(l, r, s);
-    if (l->dp <= 64) return launch_wr<64>(l, r, s);
-    if (l->dp <= 96) return launch_wr<96>(l, r, s);
-    if (l->dp <= 128) return launch_wr<128>(l, r, s);
-    return launch_wr<256>(l, r, s);
+    if (r->dt != DT_BF16 || r->n_seqs != 1 || !attn_valid(l)) return cudaErrorInvalidValue;
+    return l->exact_weights ? launch_wr_t<3>(l, r, s) : launch_wr_t<1>(l, r, s);
 }
 B2_API int b2_sizeof_mix_layer() { return (int)sizeof(MixLayer); }
 B2_API int b2_sizeof_mix_run() { return (int)sizeof(MixRun); }

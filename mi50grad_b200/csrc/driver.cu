@@ -114,15 +114,22 @@ struct ModelDesc {
     const struct MixerModelDesc* mixer;    // post-norm decoder of parallel mixers (csrc/mixers.cuh); null: the hybrid decoder above
 };
 
-// Post-norm decoders with dense bf16 / fp32 weights: x += norm1(mixer(x)), x += norm2(ff(x)).  The row, sequence,
-// logits and arg-max buffers are ModelDesc's; element-typed buffers (proj, attn_out, act, xn and the p_ forms)
-// hold bf16 or fp32 by `dt`.
-struct MixerLayerDesc {
+// Decoders with dense bf16 / fp32 weights whose layers are described one by one.  The row, sequence, logits and
+// arg-max buffers are ModelDesc's; element-typed buffers (proj, attn_out, act, xn and the p_ forms) hold bf16 or
+// fp32 by `dt`.
+//   streams == 0: post-norm, x += norm1(mixer(x)), x += norm2(ff(x));
+//   streams > 0:  pre-norm over that many residual streams joined by hyper-connections (StreamMix).
+#define MIX_PARALLEL 0            // attention beside a recurrence
+#define MIX_ATTENTION 1
+#define MIX_RECURRENCE 2
+struct MixerLayerDesc {           // one run of a layer (a layer that runs several times has several of them)
     MixLayer mix;
-    LinearDesc in_proj;           // [q | k | z | x | B | C | dt]
-    LinearDesc out_proj;          // [attention | recurrence] -> H
+    LinearDesc in_proj;           // [q | k | z | x | B | C | dt], [q | k | v] or [q | k | v | g]
+    LinearDesc out_proj;          // the mixer's columns -> H
     LinearDesc gate_up, down;     // kind LIN_NONE: no feed-forward
     const float* norm1; const float* norm2;
+    const float* hc1; const float* hc2;        // streams: StreamMix::coef behind the mixer / behind the feed-forward
+    int kind, act, act_cols, pad;              // MIX_*; ACT_* of the feed-forward; outputs of in_proj that get SiLU
 };
 struct MixerModelDesc {
     const MixerLayerDesc* layers;
@@ -134,6 +141,11 @@ struct MixerModelDesc {
     void* qbuf; void* xbc; float* dtb; float* ubuf;            // sized for max(max_rows, max_prefill) rows
     float* attn_scratch; int* attn_counters; int* ssd_counters;
     float* chunk_state; void* chunk_prev; float* chunk_decay;  // chunked scan (null: token by token only)
+    // residual streams
+    int streams, ld_embed; float embed_scale; int pad;
+    const float* hc0;             // coef of the embedding (its `in` part counts)
+    float* sx; float* p_sx;       // [rows][streams][H]
+    float* su;                    // [max_rows][H] a sublayer's input before its norm
 };
 
 // Projections queued for one chain launch, with what the stand-alone GEMV path needs to run them
@@ -737,16 +749,19 @@ static int rows_impl(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
 }
 
 // ---------------------------------------------------------------------------
-// Post-norm decoders of parallel mixers.
+// Dense-weight decoders: parts shared by both block forms, then the post-norm form.
 // ---------------------------------------------------------------------------
 static inline int mixer_rpc(const LinearDesc& L, int rows) { return rows <= DG_FMA_ROWS ? L.kslice : L.L; }
-// Decode projection; pn: the residual update its input still owes (x null), ss_out: partial sums for the next one.
+// Decode projection; pn: the residual update or norm its input still owes (x null), ss_out: partial sums for the next
+// one, sm: DG_STREAMS.
 static int mixer_gemv(Driver* d, const LinearDesc& L, const void* x, int ldx, const PostNorm& pn, int rows, void* out, int ldo,
-                      int mode, float* ss_out, float softcap, cudaStream_t s) {
+                      int mode, float* ss_out, float softcap, cudaStream_t s, int act = 0, const StreamMix* sm = nullptr) {
     DenseGemvParams p;
     memset(&p, 0, sizeof(p));
     p.w = L.w; p.x = x; p.pn = pn; p.out = out; p.ss_out = ss_out; p.ldw = L.ldw; p.ldx = ldx; p.K = L.K; p.N = L.N;
     p.rows = rows; p.ldo = ldo; p.mode = mode; p.dt = d->mx.dt; p.rpc = mixer_rpc(L, rows); p.ss_np = d->mx.ss_np; p.softcap = softcap;
+    if (mode == DG_STORE) p.act_cols = act; else p.act = act;
+    if (sm) p.sm = *sm;
     d->launches++;
     return b2_gemv_dense(&p, s);
 }
@@ -754,7 +769,7 @@ static int mixer_gemv(Driver* d, const LinearDesc& L, const void* x, int ldx, co
 // Many-row projection: tcgen05 GEMM (bf16) or the fp32 GEMM.  planes (optional, in: the most planes `out` has
 // room for, max_prefill rows apart; out: the planes written): the product may be split over K.
 static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, int T, void* out, int ldo, int mode, float softcap,
-                      cudaStream_t s, int* planes = nullptr) {
+                      cudaStream_t s, int* planes = nullptr, int act = 0) {
     d->launches++;
     const int max_ks = planes ? *planes : 1;
     if (planes) *planes = 1;
@@ -763,6 +778,7 @@ static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, in
         memset(&p, 0, sizeof(p));
         p.w = (const float*)L.w; p.x = (const float*)x; p.out = out; p.ldw = L.ldw; p.ldx = ldx; p.K = L.K; p.N = L.N; p.T = T;
         p.ldo = ldo; p.mode = mode; p.softcap = softcap;
+        if (mode == DG_STORE) p.act_cols = act; else p.act = act;
         return b2_gemm_f32(&p, s);
     }
     GemmTcParams p;
@@ -784,8 +800,9 @@ static int mixer_gemm(Driver* d, const LinearDesc& L, const void* x, int ldx, in
     p.K = L.K; p.T = T; p.t_tile = best_t > Tr ? Tr : best_t; p.k_splits = best_ks;
     p.ldo = ldo; p.out = out; p.status = d->m.tc_status; p.bf16 = 1; p.softcap = softcap;
     if (planes) { *planes = b2_gemm_tc_splits(L.K, best_ks); p.plane_stride = (long long)d->m.max_prefill * ldo; }
-    p.n_valid = mode == DG_SILU_PAIR ? L.N / 2 : L.N;
-    p.epi = mode == DG_SILU_PAIR ? TC_EPI_SILU_PAIR : (mode == DG_STORE ? TC_EPI_STORE_F16 : TC_EPI_STORE_F32);
+    p.n_valid = mode == DG_GATE_PAIR ? L.N / 2 : L.N;
+    if (mode == DG_STORE) p.act_cols = act; else p.act = act;
+    p.epi = mode == DG_GATE_PAIR ? TC_EPI_SILU_PAIR : (mode == DG_STORE ? TC_EPI_STORE_F16 : TC_EPI_STORE_F32);
     return b2_gemm_f16_tc(&p, L.w, L.ldw, x, ldx, s);
 }
 
@@ -803,6 +820,22 @@ static MixRun mixer_run(const Driver* d, bool many, int rows, int n_seqs, int fl
     r.attn_scratch = x.attn_scratch; r.attn_counters = x.attn_counters; r.ssd_counters = x.ssd_counters;
     r.chunk_state = x.chunk_state; r.chunk_prev = x.chunk_prev; r.chunk_decay = x.chunk_decay;
     return r;
+}
+
+// The kernels between a layer's in-projection and its output projection.
+static int mixer_block(Driver* d, const MixerLayerDesc& L, const MixRun& run, bool many, cudaStream_t s) {
+    const bool one = many && run.n_seqs == 1 && run.dt == DT_BF16;      // many rows of one sequence
+    MixRun r = run;
+    if (L.kind == MIX_RECURRENCE) { r.xbc = (void*)r.proj; r.ld_xbc = r.ld_proj; }     // the projection's epilogue has applied the SiLU
+    else {
+        CK(L.kind == MIX_ATTENTION ? b2_head_prepare(&L.mix, &r, s) : b2_mix_prepare(&L.mix, &r, s));
+        if (one && r.n_rows >= 16) CK(b2_window_attn_rows(&L.mix, &r, s)); else CK(b2_window_attn_decode(&L.mix, &r, s));
+        d->launches += 2;
+    }
+    if (L.kind == MIX_ATTENTION) return 0;
+    if (one && r.n_rows >= 32 && r.chunk_state) { CK(b2_ssd_chunk(&L.mix, &r, s)); d->launches += 4; }
+    else { CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2; }
+    return 0;
 }
 
 struct LayerCount {
@@ -857,13 +890,11 @@ static int mixer_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s
         const MixerLayerDesc& L = d->mlayers[li];
         LayerCount count(d, li);
         CK(project(L.in_proj, m.proj, m.ld_proj, DG_STORE));
-        CK(b2_mix_prepare(&L.mix, &r, s)); d->launches++;
-        CK(b2_window_attn_decode(&L.mix, &r, s)); d->launches++;
-        CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2;
+        CK(mixer_block(d, L, r, false, s));
         CK(mixer_gemv(d, L.out_proj, m.attn_out, m.ld_attn, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
         owed = L.norm1; owed_np = (m.H + mixer_rpc(L.out_proj, rows) - 1) / mixer_rpc(L.out_proj, rows);
         if (L.down.kind == LIN_NONE) continue;
-        CK(project(L.gate_up, m.act, x.ld_act, DG_SILU_PAIR));
+        CK(project(L.gate_up, m.act, x.ld_act, DG_GATE_PAIR));
         CK(mixer_gemv(d, L.down, m.act, x.ld_act, none, rows, x.m, m.H, DG_STORE_F32, m.ss, 0.f, s));
         owed = L.norm2; owed_np = (m.H + mixer_rpc(L.down, rows) - 1) / mixer_rpc(L.down, rows);
     }
@@ -874,40 +905,10 @@ static int mixer_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s
     return argmax_advance(d, false, rows, n_seqs, flags, s);
 }
 
-static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
+// Output head and arg-max of a many-row step (p_xn: the final-normed rows).
+static int mixer_head_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
     const ModelDesc& m = d->m;
     const MixerModelDesc& x = d->mx;
-    if (T < 1 || T > m.max_prefill) return cudaErrorInvalidValue;
-    if (flags & STEP_SPEC) return cudaErrorNotSupported;
-    d->launches = 0; d->chain_launches = 0; d->exchanges = 0;
-    CK(b2_prepare_rows(m.p_rows_tmpl, m.seqs, m.p_rows, T, nullptr, s)); d->launches++;
-    if (flags & STEP_EMBED_TOKENS)
-        CK(b2_embed_rows(m.embed, m.p_row_tokens, m.p_rows, m.seqs, m.p_h, m.p_xn, x.ld_x, T, m.H, m.vocab, x.dt, s));
-    else
-        CK(b2_post_norm(m.p_h, nullptr, nullptr, nullptr, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, 1, 0, s));
-    d->launches++;
-    const MixRun r = mixer_run(d, true, T, n_seqs, flags);
-    const bool one = n_seqs == 1 && x.dt == DT_BF16;
-    for (int li = 0; li < m.n_layers; ++li) {
-        const MixerLayerDesc& L = d->mlayers[li];
-        LayerCount count(d, li);
-        const float* after = li + 1 == m.n_layers ? x.final_norm : nullptr;      // the last update also applies the final norm
-        CK(mixer_gemm(d, L.in_proj, m.p_xn, x.ld_x, T, m.p_proj, m.ld_proj, DG_STORE, 0.f, s));
-        CK(b2_mix_prepare(&L.mix, &r, s));
-        if (one && T >= 16) CK(b2_window_attn_rows(&L.mix, &r, s)); else CK(b2_window_attn_decode(&L.mix, &r, s));
-        d->launches += 2;
-        if (one && T >= 32 && x.chunk_state) { CK(b2_ssd_chunk(&L.mix, &r, s)); d->launches += 4; }
-        else { CK(b2_ssd_step(&L.mix, &r, s)); d->launches += r.fuse_norm ? 1 : 2; }
-        int planes = x.m_planes;
-        CK(mixer_gemm(d, L.out_proj, m.p_attn, m.ld_attn, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
-        const bool ff = L.down.kind != LIN_NONE;
-        CK(b2_post_norm(m.p_h, x.p_m, L.norm1, ff ? nullptr : after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
-        if (!ff) continue;
-        CK(mixer_gemm(d, L.gate_up, m.p_xn, x.ld_x, T, m.p_act, x.ld_act, DG_SILU_PAIR, 0.f, s));
-        planes = x.m_planes;
-        CK(mixer_gemm(d, L.down, m.p_act, x.ld_act, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
-        CK(b2_post_norm(m.p_h, x.p_m, L.norm2, after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
-    }
     if (flags & STEP_HEAD_LAST) {
         if (n_seqs != 1 || (flags & STEP_ADVANCE)) return cudaErrorInvalidValue;
         PostNorm none;
@@ -923,7 +924,152 @@ static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
     return argmax_advance(d, true, T, n_seqs, flags, s);
 }
 
+static int mixer_rows(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    if (T < 1 || T > m.max_prefill) return cudaErrorInvalidValue;
+    if (flags & STEP_SPEC) return cudaErrorNotSupported;
+    d->launches = 0; d->chain_launches = 0; d->exchanges = 0;
+    CK(b2_prepare_rows(m.p_rows_tmpl, m.seqs, m.p_rows, T, nullptr, s)); d->launches++;
+    if (flags & STEP_EMBED_TOKENS)
+        CK(b2_embed_rows(m.embed, m.p_row_tokens, m.p_rows, m.seqs, m.p_h, m.p_xn, x.ld_x, T, m.H, m.vocab, x.dt, s));
+    else
+        CK(b2_post_norm(m.p_h, nullptr, nullptr, nullptr, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, 1, 0, s));
+    d->launches++;
+    const MixRun r = mixer_run(d, true, T, n_seqs, flags);
+    for (int li = 0; li < m.n_layers; ++li) {
+        const MixerLayerDesc& L = d->mlayers[li];
+        LayerCount count(d, li);
+        const float* after = li + 1 == m.n_layers ? x.final_norm : nullptr;      // the last update also applies the final norm
+        CK(mixer_gemm(d, L.in_proj, m.p_xn, x.ld_x, T, m.p_proj, m.ld_proj, DG_STORE, 0.f, s));
+        CK(mixer_block(d, L, r, true, s));
+        int planes = x.m_planes;
+        CK(mixer_gemm(d, L.out_proj, m.p_attn, m.ld_attn, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
+        const bool ff = L.down.kind != LIN_NONE;
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm1, ff ? nullptr : after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
+        if (!ff) continue;
+        CK(mixer_gemm(d, L.gate_up, m.p_xn, x.ld_x, T, m.p_act, x.ld_act, DG_GATE_PAIR, 0.f, s));
+        planes = x.m_planes;
+        CK(mixer_gemm(d, L.down, m.p_act, x.ld_act, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
+        CK(b2_post_norm(m.p_h, x.p_m, L.norm2, after, m.p_xn, x.ld_x, T, m.H, m.eps, x.dt, planes, (long long)m.max_prefill * m.H, s)); d->launches++;
+    }
+    return mixer_head_rows(d, T, n_seqs, flags, s);
+}
+
+// ---------------------------------------------------------------------------
+// Pre-norm decoders over residual streams.
+// ---------------------------------------------------------------------------
+static StreamRows stream_rows_of(const Driver* d, bool many, int rows) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    StreamRows p;
+    memset(&p, 0, sizeof(p));
+    p.sm.x = many ? x.p_sx : x.sx; p.sm.n = x.streams; p.planes = 1;
+    p.xb = many ? m.p_xn : m.xn; p.ldx = x.ld_x; p.rows = rows; p.H = m.H; p.dt = x.dt; p.eps = m.eps; p.scale = x.embed_scale;
+    return p;
+}
+static int stream_embed(Driver* d, bool many, int rows, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    StreamRows p = stream_rows_of(d, many, rows);
+    p.sm.coef = d->mx.hc0; p.w = d->mlayers[0].norm1; p.from_embedding = 1;
+    p.h = many ? m.p_h : m.h;
+    if (flags & STEP_EMBED_TOKENS) {
+        p.embed = m.embed; p.ld_embed = d->mx.ld_embed; p.vocab = m.vocab; p.row_tokens = many ? m.p_row_tokens : m.row_tokens;
+        p.meta = (const RowMeta*)(many ? m.p_rows : m.rows); p.seqs = (const SeqState*)m.seqs;
+    }
+    d->launches++;
+    return b2_stream_rows(&p, s);
+}
+// norm weights of the sublayer behind layer run li's mixer (ff: behind its feed-forward); null behind the last one
+static const float* stream_next_norm(const Driver* d, int li, bool ff) {
+    if (!ff && d->mlayers[li].down.kind != LIN_NONE) return d->mlayers[li].norm2;
+    return li + 1 < d->m.n_layers ? d->mlayers[li + 1].norm1 : nullptr;
+}
+
+// <= 8 rows.  With few rows (mixer_lazy_rows) the projection that ends a sublayer updates the streams itself and the
+// next one normalises its input while it stages it; with more rows a launch between them does both once.
+static int stream_step(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    if (rows < 1 || rows > m.max_rows || rows > B2_MAX_ROWS) return cudaErrorInvalidValue;
+    if (flags & STEP_SPEC) return cudaErrorNotSupported;
+    d->launches = 0; d->chain_launches = 0; d->exchanges = 0; d->pend.n = 0;
+    CK(b2_prepare_rows(m.rows_tmpl, m.seqs, m.rows, rows, nullptr, s)); d->launches++;
+    CK(stream_embed(d, false, rows, flags, s));
+    const bool lazy = rows <= d->mixer_lazy_rows;
+    PostNorm none, pn;
+    memset(&none, 0, sizeof(none));
+    pn = none;                                   // pn.m set: the input is still to be normalised; else it is m.xn
+    auto project = [&](const LinearDesc& L, void* out, int ldo, int mode, int act) -> int {
+        return mixer_gemv(d, L, pn.m ? nullptr : m.xn, x.ld_x, pn, rows, out, ldo, mode, nullptr, 0.f, s, act);
+    };
+    auto finish = [&](const LinearDesc& L, const void* in, int ldi, const float* coef, const float* norm) -> int {
+        pn = none;
+        if (lazy && norm) {
+            StreamMix sm;
+            memset(&sm, 0, sizeof(sm));
+            sm.x = x.sx; sm.u = x.su; sm.coef = coef; sm.n = x.streams;
+            pn.m = x.su; pn.w = norm; pn.ss = m.ss; pn.np = (m.H + mixer_rpc(L, rows) - 1) / mixer_rpc(L, rows); pn.H = m.H; pn.eps = m.eps;
+            return mixer_gemv(d, L, in, ldi, none, rows, nullptr, m.H, DG_STREAMS, m.ss, 0.f, s, 0, &sm);
+        }
+        CK(mixer_gemv(d, L, in, ldi, none, rows, x.m, m.H, DG_STORE_F32, nullptr, 0.f, s));
+        StreamRows p = stream_rows_of(d, false, rows);
+        p.sm.coef = coef; p.y = x.m; p.w = norm ? norm : x.final_norm;
+        if (!norm) p.sm.u = m.h;                 // the sum of the streams
+        d->launches++;
+        return b2_stream_rows(&p, s);
+    };
+    const MixRun r = mixer_run(d, false, rows, n_seqs, flags);
+    for (int li = 0; li < m.n_layers; ++li) {
+        const MixerLayerDesc& L = d->mlayers[li];
+        LayerCount count(d, li);
+        CK(project(L.in_proj, m.proj, m.ld_proj, DG_STORE, L.act_cols));
+        CK(mixer_block(d, L, r, false, s));
+        CK(finish(L.out_proj, m.attn_out, m.ld_attn, L.hc1, stream_next_norm(d, li, false)));
+        if (L.down.kind == LIN_NONE) continue;
+        CK(project(L.gate_up, m.act, x.ld_act, DG_GATE_PAIR, L.act));
+        CK(finish(L.down, m.act, x.ld_act, L.hc2, stream_next_norm(d, li, true)));
+    }
+    if (flags & STEP_LM_HEAD)
+        CK(mixer_gemv(d, m.lm_head, m.xn, x.ld_x, none, rows, m.logits, m.ld_logits, DG_STORE_F32, nullptr, x.softcap, s));
+    return argmax_advance(d, false, rows, n_seqs, flags, s);
+}
+
+static int stream_many(Driver* d, int T, int n_seqs, int flags, cudaStream_t s) {
+    const ModelDesc& m = d->m;
+    const MixerModelDesc& x = d->mx;
+    if (T < 1 || T > m.max_prefill) return cudaErrorInvalidValue;
+    if (flags & STEP_SPEC) return cudaErrorNotSupported;
+    d->launches = 0; d->chain_launches = 0; d->exchanges = 0;
+    CK(b2_prepare_rows(m.p_rows_tmpl, m.seqs, m.p_rows, T, nullptr, s)); d->launches++;
+    CK(stream_embed(d, true, T, flags, s));
+    auto finish = [&](const LinearDesc& L, const void* in, int ldi, const float* coef, const float* norm) -> int {
+        int planes = x.m_planes;
+        CK(mixer_gemm(d, L, in, ldi, T, x.p_m, m.H, DG_STORE_F32, 0.f, s, &planes));
+        StreamRows p = stream_rows_of(d, true, T);
+        p.sm.coef = coef; p.y = x.p_m; p.planes = planes; p.plane_stride = (long long)m.max_prefill * m.H;
+        p.w = norm ? norm : x.final_norm;
+        if (!norm) p.sm.u = m.p_h;
+        d->launches++;
+        return b2_stream_rows(&p, s);
+    };
+    const MixRun r = mixer_run(d, true, T, n_seqs, flags);
+    for (int li = 0; li < m.n_layers; ++li) {
+        const MixerLayerDesc& L = d->mlayers[li];
+        LayerCount count(d, li);
+        CK(mixer_gemm(d, L.in_proj, m.p_xn, x.ld_x, T, m.p_proj, m.ld_proj, DG_STORE, 0.f, s, nullptr, L.act_cols));
+        CK(mixer_block(d, L, r, true, s));
+        CK(finish(L.out_proj, m.p_attn, m.ld_attn, L.hc1, stream_next_norm(d, li, false)));
+        if (L.down.kind == LIN_NONE) continue;
+        CK(mixer_gemm(d, L.gate_up, m.p_xn, x.ld_x, T, m.p_act, x.ld_act, DG_GATE_PAIR, 0.f, s, nullptr, L.act));
+        CK(finish(L.down, m.p_act, x.ld_act, L.hc2, stream_next_norm(d, li, true)));
+    }
+    return mixer_head_rows(d, T, n_seqs, flags, s);
+}
+
 static int run_impl(Driver* d, int rows, int n_seqs, int flags, cudaStream_t s) {
+    if (!d->mlayers.empty() && d->mx.streams > 0)
+        return (flags & STEP_GEMM_PATH) ? stream_many(d, rows, n_seqs, flags, s) : stream_step(d, rows, n_seqs, flags, s);
     if (!d->mlayers.empty()) return (flags & STEP_GEMM_PATH) ? mixer_rows(d, rows, n_seqs, flags, s) : mixer_step(d, rows, n_seqs, flags, s);
     return (flags & STEP_GEMM_PATH) ? rows_impl(d, rows, n_seqs, flags, s) : step_impl(d, rows, n_seqs, flags, s);
 }

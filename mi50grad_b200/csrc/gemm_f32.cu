@@ -47,11 +47,11 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
     for (int i = 0; i < 4; ++i) {
         const int t = t0 + ty * 4 + i;
         if (t >= p.T) continue;
-        if (p.mode == DG_SILU_PAIR) {
+        if (p.mode == DG_GATE_PAIR) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + nl[j], o = (n >> 4) * 8 + (n & 7);
-                if (n + 8 < p.N) ((float*)p.out)[(size_t)t * p.ldo + o] = silu_p(acc[i][j]) * acc[i][j + 1];
+                if (n + 8 < p.N) ((float*)p.out)[(size_t)t * p.ldo + o] = (p.act == ACT_RELU ? fmaxf(acc[i][j], 0.f) : silu_p(acc[i][j])) * acc[i][j + 1];
             }
         } else {
 #pragma unroll
@@ -60,7 +60,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
                 if (n < p.N) {
                     const float v = acc[i][j];
                     ((float*)p.out)[(size_t)t * p.ldo + n] =
-                        (p.mode == DG_STORE_F32 && p.softcap > 0.f) ? p.softcap * tanhf(v / p.softcap) : v;
+                        (p.mode == DG_STORE_F32 && p.softcap > 0.f) ? p.softcap * tanhf(v / p.softcap)
+                                                                    : (p.mode == DG_STORE && n < p.act_cols ? silu_p(v) : v);
                 }
             }
         }
@@ -69,7 +70,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
 
 B2_API int b2_gemm_f32(const GemmF32Params* p, cudaStream_t s) {
     if (p->T < 1 || p->N < 1 || p->K < 1 || p->ldx < p->K || p->ldw < p->K) return cudaErrorInvalidValue;
-    if (p->mode == DG_SILU_PAIR && (p->N & 15)) return cudaErrorInvalidValue;
+    if (p->mode == DG_GATE_PAIR && (p->N & 15)) return cudaErrorInvalidValue;
     dim3 grid((p->N + GF_T - 1) / GF_T, (p->T + GF_T - 1) / GF_T);
     return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, s, *p);
 }

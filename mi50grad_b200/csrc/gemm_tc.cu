@@ -262,7 +262,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                         float up = __shfl_down_sync(0xffffffffu, v, 8);
                         int tt = t0 + c0 + c;
                         if (is_gate && c0 + c < Tp && tt < p.T && o < p.n_valid)
-                            tc_store16(p, (size_t)tt * p.ldo + o, silu_f(v) * up);
+                            tc_store16(p, (size_t)tt * p.ldo + o, (p.act ? fmaxf(v, 0.f) : silu_f(v)) * up);
                     }
                 } else if (p.epi == TC_EPI_PUSH_F32) {
                     // plain stores into the owner's memory over NVLink (posted writes, 128 bytes per warp)
@@ -284,7 +284,7 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                         if (c0 + c < Tp && tt < p.T && n < p.n_valid) {
                             float v = __uint_as_float(r[c]);
                             size_t o = (size_t)tt * p.ldo + n;
-                            if (p.epi == TC_EPI_STORE_F16) tc_store16(p, o, v);
+                            if (p.epi == TC_EPI_STORE_F16) tc_store16(p, o, n < p.act_cols ? silu_f(v) : v);
                             else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o + plane] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
                             else if (gridDim.z > 1) atomicAdd((float*)p.out + o, v);     // split-K partial
                             else ((float*)p.out)[o] += v;

@@ -39,6 +39,8 @@ struct GemmTcParams {
     float softcap;           // TC_EPI_STORE_F32: > 0 stores softcap * tanh(y / softcap)
     long long plane_stride;  // floats between the planes of a split-K TC_EPI_STORE_F32
     int box_rows;            // set by the launcher: token rows per TMA load
+    int act;                 // TC_EPI_SILU_PAIR: 1 = relu(gate) * up instead of silu(gate) * up
+    int act_cols;            // TC_EPI_STORE_F16: SiLU on the outputs n < act_cols
     int pad3;
 };
 

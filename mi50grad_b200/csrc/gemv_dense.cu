@@ -15,7 +15,9 @@
 // The input is either an activation row, or the residual stream together with the raw output of the
 // sublayer before it (PostNorm): every CTA forms x = h + norm(m) * w while it stages its input, and the
 // CTAs share out storing the updated stream.  That removes the serial "normalise and add" launch of a
-// post-norm block.
+// post-norm block.  In a pre-norm block with several residual streams the projection that ends a sublayer updates
+// the streams in its epilogue and leaves the next sublayer's input with partial sums of squares; the next
+// projection normalises it while it stages (PostNorm without h).
 #include "mixers.cuh"
 
 #define DG_THREADS 256
@@ -58,6 +60,12 @@ __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const 
     const size_t o = (size_t)m * n.H + k;
     const bool mine = (k >> 2) % (int)gridDim.x == (int)blockIdx.x;
     if ((n.H & 3) == 0) {
+        if (!n.h) {
+            const float4 m4 = *(const float4*)(n.m + o), w4 = *(const float4*)(n.w + k);
+            const float iv = inv[m];
+            v[0] = m4.x * iv * w4.x; v[1] = m4.y * iv * w4.y; v[2] = m4.z * iv * w4.z; v[3] = m4.w * iv * w4.w;
+            return;
+        }
         const float4 h4 = *(const float4*)(n.h + o);
         v[0] = h4.x; v[1] = h4.y; v[2] = h4.z; v[3] = h4.w;
         if (n.m) {
@@ -71,6 +79,7 @@ __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const 
         for (int e = 0; e < 4; ++e) {
             v[e] = 0.f;
             if (k + e < n.H) {
+                if (!n.h) { v[e] = n.m[o + e] * inv[m] * n.w[k + e]; continue; }
                 v[e] = n.h[o + e];
                 if (n.m) { v[e] += n.m[o + e] * inv[m] * n.w[k + e]; if (mine) n.hout[o + e] = v[e]; }
             }
@@ -80,13 +89,14 @@ __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const 
 
 // Finished [rpc][8] tile in y_s -> output (both element types).
 template <typename T>
-__device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, const float (*y_s)[8], int tid, int lane, int warp) {
+__device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, float (*y_s)[8], int tid, int lane, int warp) {
     const int n0 = blockIdx.x * p.rpc;
-    if (p.mode == DG_SILU_PAIR) {
+    if (p.mode == DG_GATE_PAIR) {
         const int half = p.rpc >> 1;
         for (int i = tid; i < half * p.rows; i += DG_THREADS) {
             const int m = i / half, j = i % half, nl = (j >> 3) * 16 + (j & 7), o = blockIdx.x * half + j;
-            if (2 * o < p.N) ((T*)p.out)[(size_t)m * p.ldo + o] = to_t<T>(silu_p(y_s[nl][m]) * y_s[nl + 8][m]);
+            const float g = y_s[nl][m];
+            if (2 * o < p.N) ((T*)p.out)[(size_t)m * p.ldo + o] = to_t<T>((p.act == ACT_RELU ? fmaxf(g, 0.f) : silu_p(g)) * y_s[nl + 8][m]);
         }
         return;
     }
@@ -94,10 +104,15 @@ __device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, const floa
         const int m = i / p.rpc, nl = i % p.rpc, n = n0 + nl;
         if (n >= p.N) continue;
         const float v = y_s[nl][m];
-        if (p.mode == DG_STORE) ((T*)p.out)[(size_t)m * p.ldo + n] = to_t<T>(v);
-        else ((float*)p.out)[(size_t)m * p.ldo + n] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
+        if (p.mode == DG_STORE) ((T*)p.out)[(size_t)m * p.ldo + n] = to_t<T>(n < p.act_cols ? silu_p(v) : v);
+        else if (p.mode == DG_STREAMS) {
+            float y[1] = {v};
+            stream_mix<1>(p.sm.n, p.sm.x + (size_t)m * p.sm.n * p.N + n, p.sm.coef, p.N, y);
+            p.sm.u[(size_t)m * p.N + n] = y_s[nl][m] = y[0];
+        } else ((float*)p.out)[(size_t)m * p.ldo + n] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
     }
-    if (p.mode == DG_STORE_F32 && p.ss_out && warp < p.rows) {
+    if (p.mode == DG_STREAMS) __syncthreads();
+    if (p.mode >= DG_STORE_F32 && p.ss_out && warp < p.rows) {
         float s = 0.f;
         for (int nl = lane; nl < p.rpc; nl += 32) if (n0 + nl < p.N) s += y_s[nl][warp] * y_s[nl][warp];
         s = warp_sum(s);
@@ -360,8 +375,9 @@ static int launch_dg(const DenseGemvParams* p, cudaStream_t s) {
 B2_API int b2_gemv_dense(const DenseGemvParams* p, cudaStream_t s) {
     if (p->rows < 1 || p->rows > B2_MAX_ROWS || p->K < 1 || p->N < 1 || (p->ldw & 7) || p->ldw < p->K || ((uintptr_t)p->w & 15))
         return cudaErrorInvalidValue;
-    if (p->mode == DG_SILU_PAIR && (p->rpc < 16 || (p->N & 15))) return cudaErrorInvalidValue;
-    if (p->x ? (p->ldx < p->K || ((uintptr_t)p->x & 15)) : (!p->pn.h || p->pn.H != p->K)) return cudaErrorInvalidValue;
+    if (p->mode == DG_GATE_PAIR && (p->rpc < 16 || (p->N & 15))) return cudaErrorInvalidValue;
+    if (p->x ? (p->ldx < p->K || ((uintptr_t)p->x & 15)) : ((!p->pn.h && !p->pn.m) || p->pn.H != p->K)) return cudaErrorInvalidValue;
+    if (p->mode == DG_STREAMS && (p->sm.n < 1 || p->sm.n > STREAMS_MAX || !p->sm.x || !p->sm.u || !p->sm.coef)) return cudaErrorInvalidValue;
     if (p->ss_out && (p->N + p->rpc - 1) / p->rpc > p->ss_np) return cudaErrorInvalidValue;
     const bool tc = p->dt == DT_BF16 && (p->mma || p->rows > DG_FMA_ROWS);
     if (tc) {

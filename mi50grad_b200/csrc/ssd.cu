@@ -1,7 +1,9 @@
-// Mamba-2 (state-space duality) recurrence of a parallel mixer:
-//     S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T,     y_t = S_t^T C_t + D x_t
-// with S [N x P] fp32 per head, B and C shared by the heads of a group, followed by
-// u = y * silu(z) and an RMSNorm of u in ngroups equal parts.
+// Linear recurrences with a scalar decay per head and token:
+//     S_t = a_t S_(t-1) + dt_t B_t x_t^T,     y_t = S_t^T C_t + D x_t
+// with S [N x P] fp32 per head, B and C shared by the heads of a group.
+//   Mamba-2 (state-space duality): a_t = exp(-exp(A_log) dt_t); then an RMSNorm of y * silu(z) in ngroups parts.
+//   Lightning attention: a constant per head, dt = 1, no D, q / k / v in the places of C / B / x, every head its own
+//   group; then an RMSNorm of y times sigmoid(z).
 //
 //   ssd_step    token by token: one CTA per (head, 32 columns of P, sequence), the state in registers
 //               (requested before the dependency wait); the last CTA of a norm part normalises it.
@@ -17,6 +19,7 @@ template <typename T>
 __device__ __forceinline__ void conv_history(const MixLayer& L, const MixRun& R, int seq, int r0, int r1, int c0, int c1,
                                              int tid, int nthr) {
     const int C = L.heads * L.P + 2 * L.groups * L.N, K = L.taps - 1, n = r1 - r0;
+    if (K == 0) return;
     T* hist = (T*)L.conv_state + (size_t)seq * K * C;
     for (int c = c0 + tid; c < c1; c += nthr)
         for (int i = 0; i < K; ++i) {
@@ -39,23 +42,68 @@ __device__ __forceinline__ void conv_history_of(const MixLayer& L, const MixRun&
     }
 }
 
-// RMSNorm of one part of one row: out = u / rms(u) * w * right_scale, into the columns behind the attention's.
+__device__ __forceinline__ uint32_t sc_pack(bf16 a, bf16 b) {
+    return (uint32_t)__bfloat16_as_ushort(a) | ((uint32_t)__bfloat16_as_ushort(b) << 16);
+}
+// log decay and step size of the token in row r
+__device__ __forceinline__ float rec_rate(const MixLayer& L, int h) { return L.decay ? L.log_decay[h] : -expf(L.A_log[h]); }
+__device__ __forceinline__ float rec_dt(const MixLayer& L, const MixRun& R, int r, int h) {
+    return L.decay ? 1.f : R.dtb[(size_t)r * R.ld_dt + h];
+}
+
+// RMSNorm of one part of one row: out = u / rms(u) * w * right_scale (* sigmoid(z)), from column out_col on.
+#define NP_REGS 4                // float4s per thread that stay in registers between the passes
 template <typename T>
 __device__ __forceinline__ void norm_part(const MixLayer& L, const MixRun& R, int r, int part, float* red) {
-    const int I = L.heads * L.P, w = I / L.ngroups, c0 = part * w, tid = threadIdx.x;
+    const int I = L.heads * L.P, w = I / L.ngroups, c0 = part * w, tid = threadIdx.x, nt = blockDim.x;
     const float* u = R.ubuf + (size_t)r * R.ld_u + c0;
-    T* out = (T*)R.out + (size_t)r * R.ldo + L.H * L.d + c0;
-    float v[4], ss = 0.f;
+    const float* nw = L.norm_w + c0;
+    T* out = (T*)R.out + (size_t)r * R.ldo + L.out_col + c0;
+    const T* z = (const T*)R.proj + (size_t)r * R.ld_proj + L.off_z + c0;
+    const bool gate = L.gate == REC_NORM_SIGMOID;
+    auto one = [&](int i, float v, float inv) {
+        v *= inv * nw[i] * L.right_scale;
+        out[i] = to_t<T>(gate ? v * sigmoid_p(ld_f(z + i)) : v);
+    };
+    float ss = 0.f;
+    if (((w | c0 | R.ld_u) & 3) == 0) {
+        float4 v[NP_REGS];
+        const int w4 = w >> 2;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) { const int i = tid + j * blockDim.x; v[j] = i < w ? __ldcg(u + i) : 0.f; ss += v[j] * v[j]; }
-    for (int i = tid + 4 * blockDim.x; i < w; i += blockDim.x) { const float x = __ldcg(u + i); ss += x * x; }
-    const float inv = rsqrtf(block_sum(ss, red) / (float)w + L.eps);
+        for (int j = 0; j < NP_REGS; ++j) {
+            const int i = tid + j * nt;
+            v[j] = i < w4 ? __ldcg((const float4*)u + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-        const int i = tid + j * blockDim.x;
-        if (i < w) out[i] = to_t<T>(v[j] * inv * L.norm_w[c0 + i] * L.right_scale);
+        for (int j = 0; j < NP_REGS; ++j) ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+        for (int i = tid + NP_REGS * nt; i < w4; i += nt) {
+            const float4 q = __ldcg((const float4*)u + i);
+            ss += q.x * q.x + q.y * q.y + q.z * q.z + q.w * q.w;
+        }
+        const float inv = rsqrtf(block_sum(ss, red) / (float)w + L.eps);
+        const bool packed = sizeof(T) == 2 && (((int)R.ldo | L.out_col | R.ld_proj | L.off_z) & 3) == 0;
+        auto four = [&](int i, const float4& q) {
+            if (packed) {
+                const float4 w = ((const float4*)nw)[i];
+                const float f = inv * L.right_scale;
+                float o[4] = {q.x * f * w.x, q.y * f * w.y, q.z * f * w.z, q.w * f * w.w};
+                if (gate) {
+                    const uint2 g = *(const uint2*)(z + 4 * i);
+                    o[0] *= sigmoid_p(__uint_as_float(g.x << 16)); o[1] *= sigmoid_p(__uint_as_float(g.x & 0xffff0000u));
+                    o[2] *= sigmoid_p(__uint_as_float(g.y << 16)); o[3] *= sigmoid_p(__uint_as_float(g.y & 0xffff0000u));
+                }
+                uint2 pk; pk.x = sc_pack(__float2bfloat16(o[0]), __float2bfloat16(o[1])); pk.y = sc_pack(__float2bfloat16(o[2]), __float2bfloat16(o[3]));
+                *(uint2*)(out + 4 * i) = pk;
+            } else { one(4 * i, q.x, inv); one(4 * i + 1, q.y, inv); one(4 * i + 2, q.z, inv); one(4 * i + 3, q.w, inv); }
+        };
+#pragma unroll
+        for (int j = 0; j < NP_REGS; ++j) if (tid + j * nt < w4) four(tid + j * nt, v[j]);
+        for (int i = tid + NP_REGS * nt; i < w4; i += nt) four(i, __ldcg((const float4*)u + i));
+        return;
     }
-    for (int i = tid + 4 * blockDim.x; i < w; i += blockDim.x) out[i] = to_t<T>(__ldcg(u + i) * inv * L.norm_w[c0 + i] * L.right_scale);
+    for (int i = tid; i < w; i += nt) { const float x = __ldcg(u + i); ss += x * x; }
+    const float inv = rsqrtf(block_sum(ss, red) / (float)w + L.eps);
+    for (int i = tid; i < w; i += nt) one(i, __ldcg(u + i), inv);
 }
 
 template <typename T>
@@ -79,7 +127,7 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_step_kernel(const MixLayer L, 
     pdl_launch_dependents();
     const int h = blockIdx.x, p0 = blockIdx.y * 32, sq = blockIdx.z;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int I = L.heads * L.P, grp = h / (L.heads / L.groups), p = p0 + lane;
+    const int grp = h / (L.heads / L.groups), p = p0 + lane;
     const bool pv = p < L.P;
     const int r0 = R.seq_rows[sq], r1 = R.seq_rows[sq + 1];
     const int seq = R.rows[r0].seq;
@@ -88,18 +136,19 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_step_kernel(const MixLayer L, 
     float st[NB];
 #pragma unroll
     for (int i = 0; i < NB; ++i) { const int n = warp + SS_WARPS * i; st[i] = (pv && n < L.N) ? S[(size_t)n * L.P] : 0.f; }
-    const float A = -expf(L.A_log[h]), Dh = L.D[h];
+    const float A = rec_rate(L, h), Dh = L.D ? L.D[h] : 0.f, a_const = L.decay ? L.decay[h] : 0.f;
+    const bool gated = L.gate == REC_GATE_SILU_NORM;
     pdl_wait();
     for (int r = r0; r < r1; ++r) {
         const T* xbc = (const T*)R.xbc + (size_t)r * R.ld_xbc;
         for (int n = tid; n < SS_WARPS * NB; n += SS_THREADS) {
-            Bs[n] = n < L.N ? ld_f(xbc + I + grp * L.N + n) : 0.f;
-            Cs[n] = n < L.N ? ld_f(xbc + I + (L.groups + grp) * L.N + n) : 0.f;
+            Bs[n] = n < L.N ? ld_f(xbc + L.rB + grp * L.N + n) : 0.f;
+            Cs[n] = n < L.N ? ld_f(xbc + L.rC + grp * L.N + n) : 0.f;
         }
-        const float x = pv ? ld_f(xbc + h * L.P + p) : 0.f;
-        const float dt = R.dtb[(size_t)r * R.ld_dt + h];
-        const float z = (warp == 0 && pv) ? ld_f((const T*)R.proj + (size_t)r * R.ld_proj + L.off_z + h * L.P + p) : 0.f;
-        const float a = expf(A * dt), dx = dt * x;
+        const float x = pv ? ld_f(xbc + L.rx + h * L.P + p) : 0.f;
+        const float dt = rec_dt(L, R, r, h);
+        const float z = (gated && warp == 0 && pv) ? ld_f((const T*)R.proj + (size_t)r * R.ld_proj + L.off_z + h * L.P + p) : 0.f;
+        const float a = L.decay ? a_const : expf(A * dt), dx = dt * x;
         __syncthreads();
         float y = 0.f;
 #pragma unroll
@@ -114,7 +163,7 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_step_kernel(const MixLayer L, 
             float s = 0.f;
 #pragma unroll
             for (int w = 0; w < SS_WARPS; ++w) s += part[w][lane];
-            R.ubuf[(size_t)r * R.ld_u + h * L.P + p] = (s + Dh * x) * silu_p(z);
+            R.ubuf[(size_t)r * R.ld_u + h * L.P + p] = (s + Dh * x) * (gated ? silu_p(z) : 1.f);
         }
     }
     if (R.commit) {
@@ -142,7 +191,7 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_step_kernel(const MixLayer L, 
 
 static bool ssd_valid(const MixLayer* l) {
     return l->heads >= 1 && l->P >= 1 && l->N >= 1 && l->N <= 256 && l->groups >= 1 && l->heads % l->groups == 0 &&
-           l->ngroups >= 1 && (l->heads * l->P) % l->ngroups == 0 && l->taps >= 1;
+           l->ngroups >= 1 && (l->heads * l->P) % l->ngroups == 0 && l->taps >= 1 && (l->decay ? l->log_decay != nullptr : l->A_log != nullptr);
 }
 
 template <typename T>
@@ -188,14 +237,11 @@ __device__ __forceinline__ void sc_split(float v, bf16 (&t)[SC_TERMS]) {
 #pragma unroll
     for (int i = 0; i < SC_TERMS; ++i) { t[i] = __float2bfloat16(v); v -= __bfloat162float(t[i]); }
 }
-__device__ __forceinline__ uint32_t sc_pack(bf16 a, bf16 b) {
-    return (uint32_t)__bfloat16_as_ushort(a) | ((uint32_t)__bfloat16_as_ushort(b) << 16);
-}
 
 // cumulative log decay of a chunk (one warp; two tokens per lane)
-__device__ __forceinline__ void sc_cumsum(const MixRun& R, int t0, int n, int h, float A, float* la, float* dts, int lane) {
-    const float d0 = 2 * lane < n ? R.dtb[(size_t)(t0 + 2 * lane) * R.ld_dt + h] : 0.f;
-    const float d1 = 2 * lane + 1 < n ? R.dtb[(size_t)(t0 + 2 * lane + 1) * R.ld_dt + h] : 0.f;
+__device__ __forceinline__ void sc_cumsum(const MixLayer& L, const MixRun& R, int t0, int n, int h, float A, float* la, float* dts, int lane) {
+    const float d0 = 2 * lane < n ? rec_dt(L, R, t0 + 2 * lane, h) : 0.f;
+    const float d1 = 2 * lane + 1 < n ? rec_dt(L, R, t0 + 2 * lane + 1, h) : 0.f;
     const float a0 = A * d0, a1 = A * d1;
     float s = a0 + a1;
 #pragma unroll
@@ -230,18 +276,18 @@ __global__ void __launch_bounds__(128) ssd_chunk_state_kernel(const MixLayer L, 
     pdl_launch_dependents();
     const int c = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * SC_P;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int I = L.heads * L.P, grp = h / (L.heads / L.groups), pw = min(SC_P, L.P - p0);
+    const int grp = h / (L.heads / L.groups), pw = min(SC_P, L.P - p0);
     const int t0 = c * SC_T, n = min(SC_T, R.n_rows - t0);
-    const float A = -expf(L.A_log[h]);
+    const float A = rec_rate(L, h);
     pdl_wait();
-    sc_stage(R, t0, n, I + grp * L.N, L.N, Np, Bs, LDN, tid, 128);
-    if (warp == 0) sc_cumsum(R, t0, n, h, A, la, dts, lane);
+    sc_stage(R, t0, n, L.rB + grp * L.N, L.N, Np, Bs, LDN, tid, 128);
+    if (warp == 0) sc_cumsum(L, R, t0, n, h, A, la, dts, lane);
     __syncthreads();
     const float end = la[SC_T - 1];
     for (int i = tid; i < SC_T * SC_P; i += 128) {
         const int s = i / SC_P, p = i % SC_P;
         float v = 0.f;
-        if (s < n && p < pw) v = ld_f((const bf16*)R.xbc + (size_t)(t0 + s) * R.ld_xbc + h * L.P + p0 + p) * (dts[s] * expf(end - la[s]));
+        if (s < n && p < pw) v = ld_f((const bf16*)R.xbc + (size_t)(t0 + s) * R.ld_xbc + L.rx + h * L.P + p0 + p) * (dts[s] * expf(end - la[s]));
         bf16 q[SC_TERMS];
         sc_split(v, q);
 #pragma unroll
@@ -330,13 +376,14 @@ __global__ void __launch_bounds__(128) ssd_chunk_out_kernel(const MixLayer L, co
     pdl_launch_dependents();
     const int c = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * SC_P;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int I = L.heads * L.P, grp = h / (L.heads / L.groups), pw = min(SC_P, L.P - p0), pwp = (pw + 7) & ~7;
+    const int grp = h / (L.heads / L.groups), pw = min(SC_P, L.P - p0), pwp = (pw + 7) & ~7;
     const int t0 = c * SC_T, n = min(SC_T, R.n_rows - t0);
-    const float A = -expf(L.A_log[h]), Dh = L.D[h];
+    const float A = rec_rate(L, h), Dh = L.D ? L.D[h] : 0.f;
+    const bool gated = L.gate == REC_GATE_SILU_NORM;
     pdl_wait();
-    sc_stage(R, t0, n, I + (L.groups + grp) * L.N, L.N, Np, Cs, LDN, tid, 128);
-    sc_stage(R, t0, n, I + grp * L.N, L.N, Np, Bs, LDN, tid, 128);
-    sc_stage(R, t0, n, h * L.P + p0, pw, SC_P, Xs, SC_LDP, tid, 128);
+    sc_stage(R, t0, n, L.rC + grp * L.N, L.N, Np, Cs, LDN, tid, 128);
+    sc_stage(R, t0, n, L.rB + grp * L.N, L.N, Np, Bs, LDN, tid, 128);
+    sc_stage(R, t0, n, L.rx + h * L.P + p0, pw, SC_P, Xs, SC_LDP, tid, 128);
     {
         const bf16* src = (const bf16*)R.chunk_prev + ((size_t)c * L.heads + h) * SC_TERMS * L.N * Pp + p0;
         const int ppr = SC_P / 8;
@@ -348,7 +395,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_out_kernel(const MixLayer L, co
         }
         cp_async_commit();
     }
-    if (warp == 0) sc_cumsum(R, t0, n, h, A, la, dts, lane);
+    if (warp == 0) sc_cumsum(L, R, t0, n, h, A, la, dts, lane);
     cp_async_wait<0>();
     __syncthreads();
     if (warp * 16 >= n) return;
@@ -421,8 +468,9 @@ __global__ void __launch_bounds__(128) ssd_chunk_out_kernel(const MixLayer L, co
         for (int e = 0; e < 4; ++e) {
             const int r = e >= 2 ? r_hi : r_lo, p = 8 * j + 2 * t + (e & 1);
             if (r < n && p < pw) {
-                const float z = ld_f((const bf16*)R.proj + (size_t)(t0 + r) * R.ld_proj + L.off_z + h * L.P + p0 + p);
-                R.ubuf[(size_t)(t0 + r) * R.ld_u + h * L.P + p0 + p] = (o[j][e] + Dh * ld_f(Xs + r * SC_LDP + p)) * silu_p(z);
+                float u = o[j][e] + Dh * ld_f(Xs + r * SC_LDP + p);
+                if (gated) u *= silu_p(ld_f((const bf16*)R.proj + (size_t)(t0 + r) * R.ld_proj + L.off_z + h * L.P + p0 + p));
+                R.ubuf[(size_t)(t0 + r) * R.ld_u + h * L.P + p0 + p] = u;
             }
         }
 }

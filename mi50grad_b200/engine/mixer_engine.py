@@ -1,12 +1,15 @@
-"""Engine of the post-norm decoders of parallel mixers (Degedra) on one GPU.
+"""Engine of the decoders whose layers are described one by one, on one GPU: the
+post-norm decoder of parallel mixers (Degedra) here, the pre-norm decoder over
+residual streams (Vekerax) in `vekerax_engine`, which replaces only what a layer is
+made of.
 
 The token-level interface, the row templates, the graph-captured decode step and the
 C++ driver are those of `InferenceEngine`; what differs is what the driver is given:
 dense bf16 (or, for a model run entirely in 32 bits, fp32) projections fused per
-layer, per-layer caches and recurrent states (`MixerStates`), and the work buffers of
-the mixer kernels.
+layer, caches and recurrent states of every run of a layer (`MixerStates`), and the
+work buffers of the mixer kernels.
 
-Fusions made when weights are loaded:
+Fusions made when weights are loaded (Degedra):
 * [q | k | right.in] is one in-projection, so both branches of the mixer come from one
   launch;
 * the branches' output projections are one matrix over the concatenation
@@ -24,7 +27,7 @@ from typing import Dict, List, Optional, Sequence, Union
 import numpy as np
 import torch
 
-from ..config import DegedraConfig, EngineConfig
+from ..config import EngineConfig, WindowAttentionSpec
 from ..models.mixer_weights import MixerLayerWeights, MixerModelWeights, random_mixer_model
 from ..ops import lib as L
 from .engine import InferenceEngine
@@ -67,6 +70,15 @@ class MixerLinear:
         return self.w.numel() * self.w.element_size()
 
 
+def fill_attention(m: L.MixLayer, a: WindowAttentionSpec, k: torch.Tensor, v: torch.Tensor, off_q: int, separate_values: bool):
+    """Sizes, constants, caches and projection columns [q | k (| v)] of an attention."""
+    m.H, m.G, m.d, m.dp, m.rot, m.window = a.heads, a.kv_heads, a.dim, _up8(a.dim), a.rot_dims, a.window
+    m.dv, m.vp, m.head_norm, m.keep_first, m.softcap = a.vd, _up8(a.vd), int(a.head_norm), a.keep_first, a.softcap
+    m.attn_scale, m.kcache, m.vcache = a.scale, k.data_ptr(), v.data_ptr()
+    m.off_q, m.off_k = off_q, off_q + a.heads * a.dim
+    m.off_v = m.off_k + a.kv_heads * a.dim if separate_values else -1
+
+
 def interleave_dense_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     """[F, K] x 2 -> [2 * F', K] with rows g0..g7 u0..u7 g8.. (F' = F padded to 8 with zero rows)."""
     F, K = gate.shape
@@ -82,7 +94,7 @@ def interleave_dense_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tens
 class MixerLayer:
     """Device weights of one layer (shared by layers that use another's tensors)."""
 
-    def __init__(self, eng: "MixerEngine", lw: MixerLayerWeights):
+    def __init__(self, eng: "MixerEngine", lw: MixerLayerWeights, layer_idx: int):
         dev, f32 = eng.device, eng._f32
         t = lambda w: w.to(device=dev, dtype=eng.dtype)
         lin = lambda w, pair=False: MixerLinear(w, eng.lin_kind, eng.dtype, dev, pair)
@@ -102,16 +114,24 @@ class MixerLayer:
 
 
 class MixerEngine(InferenceEngine):
-    def __init__(self, config: DegedraConfig, device_id: int = 0, max_seq_len: int = 2048, dtype: str = "bfloat16",
+    """`layer_type`, `weights_type` and the methods `_mix_layer`, `_layer_desc`, `_extend_model` are what an
+    architecture of this kind replaces."""
+    layer_type = MixerLayer
+    weights_type = MixerLayerWeights
+
+    def __init__(self, config, device_id: int = 0, max_seq_len: int = 2048, dtype: str = "bfloat16",
                  engine_config: Optional[EngineConfig] = None, max_batch: int = 1):
         if dtype not in DTYPES:
             raise ValueError(f"dtype must be one of {sorted(DTYPES)}")
         if not torch.cuda.is_available():
-            raise RuntimeError("MixerEngine needs a CUDA device")
+            raise RuntimeError(f"{type(self).__name__} needs a CUDA device")
         self.dtype_name = dtype
         self.dtype, self.dt, self.lin_kind = DTYPES[dtype]
         self._init_common(config, device_id, max_seq_len, 1, 0, engine_config, None, max_batch)
         self.spec = SimpleNamespace(vocab=(0, config.vocab_size), vocab_local=config.vocab_size)
+        self.runs = config.run_order()               # layer of every run of a layer in a step
+        if not self.runs:
+            raise ValueError("the model runs no layer")
         self.states = MixerStates(config, max_seq_len, max_batch, self.device, self.dtype)
         self.use_tc_prefill = True       # many rows have a path of their own in both element types
         self._shared: Dict[int, MixerLayer] = {}
@@ -121,16 +141,19 @@ class MixerEngine(InferenceEngine):
     def _f32(self, t: torch.Tensor) -> torch.Tensor:
         return t.to(device=self.device, dtype=torch.float32).contiguous()
 
+    def _weight_layer(self, i: int) -> int:
+        return self.config.weight_layer(i)
+
     def load_layer_weights(self, layer_idx: int, lw: Union[MixerLayerWeights, dict]):
         """A layer that uses another layer's tensors gets that layer's device weights, whichever of them is
         loaded first."""
         if isinstance(lw, dict):
-            lw = MixerLayerWeights(**lw)
-        j = self.config.weight_layer(layer_idx)
+            lw = self.weights_type(**lw)
+        j = self._weight_layer(layer_idx)
         if j == layer_idx or j not in self._shared:
-            self._shared[j] = MixerLayer(self, lw)
+            self._shared[j] = self.layer_type(self, lw, layer_idx)
             for i in range(len(self.layers)):
-                if self.layers[i] is not None and self.config.weight_layer(i) == j:
+                if self.layers[i] is not None and self._weight_layer(i) == j:
                     self.layers[i] = self._shared[j]
         self.layers[layer_idx] = self._shared[j]
         self._drop_driver()
@@ -149,10 +172,10 @@ class MixerEngine(InferenceEngine):
 
     def load_model(self, mw: MixerModelWeights):
         for i, lw in enumerate(mw.layers):
-            if self.config.weight_layer(i) == i:
+            if self._weight_layer(i) == i:
                 self.load_layer_weights(i, lw)
         for i, lw in enumerate(mw.layers):
-            if self.config.weight_layer(i) != i:
+            if self._weight_layer(i) != i:
                 self.load_layer_weights(i, lw)
         self.load_embedding(mw.embed)
         self.load_lm_head(mw.head)
@@ -162,8 +185,8 @@ class MixerEngine(InferenceEngine):
         self.load_model(random_mixer_model(self.config, seed, self.device, self.dtype))
 
     def weight_bytes(self) -> int:
-        """Bytes one decode step streams (a shared layer counts every time it runs)."""
-        return sum(l.nbytes() for ly in self.layers for l in ly.linears()) + self.lm_head.nbytes()
+        """Bytes one decode step streams (a layer counts every time it runs)."""
+        return sum(l.nbytes() for i in self.runs for l in self.layers[i].linears()) + self.lm_head.nbytes()
 
     def _rope_tables(self, base: float, rot: int):
         key = (base, rot)
@@ -174,27 +197,38 @@ class MixerEngine(InferenceEngine):
         return self._rope[key]
 
     # ------------------------------------------------------------------ driver
-    def _mix_layer(self, i: int) -> L.MixLayer:
-        """Layer i's sizes, constants and pointers for the mixer kernels."""
+    def _mix_layer(self, run: int) -> L.MixLayer:
+        """Sizes, constants and pointers of run `run` of a layer for the mixer kernels."""
+        i = self.runs[run]
         l, dl, st = self.config.layers[i], self.layers[i], self.states
         a, s = l.attention, l.ssd
         m = L.MixLayer()
-        m.H, m.G, m.d, m.dp, m.rot, m.window = a.heads, a.kv_heads, a.dim, _up8(a.dim), a.rot_dims, a.window
-        m.attn_scale, m.left_scale, m.right_scale, m.eps = a.scale, l.left_scale, l.right_scale, self.config.rms_norm_eps
+        fill_attention(m, a, st.k[run], st.v[run], 0, False)
+        m.left_scale, m.right_scale, m.eps = l.left_scale, l.right_scale, self.config.rms_norm_eps
         m.q_norm, m.k_norm = dl.q_norm.data_ptr(), dl.k_norm.data_ptr()
         cos, sin = self._rope_tables(a.rot_base, a.rot_dims)
         m.cos_tab, m.sin_tab = cos.data_ptr(), sin.data_ptr()
-        m.kcache, m.vcache = st.k[i].data_ptr(), st.v[i].data_ptr()
         m.heads, m.P, m.N, m.groups, m.ngroups, m.taps = s.heads, s.vdim, s.state, s.groups, s.norm_groups, s.conv
         m.conv_w, m.conv_b, m.dt_bias = dl.conv.data_ptr(), dl.conv_b.data_ptr(), dl.dt_bias.data_ptr()
         m.A_log, m.D, m.norm_w = dl.A_log.data_ptr(), dl.D.data_ptr(), dl.ssd_norm.data_ptr()
-        m.state, m.conv_state = st.S[i].data_ptr(), st.conv[i].data_ptr()
-        m.off_q, m.off_k = 0, a.heads * a.dim
+        m.state, m.conv_state = st.S[run].data_ptr(), st.conv[run].data_ptr()
         m.off_z = m.off_k + a.kv_heads * a.dim
         m.off_x = m.off_z + s.inner
         m.off_dt = m.off_x + s.conv_channels
+        m.rx, m.rB, m.rC = 0, s.inner, s.inner + s.groups * s.state
+        m.gate, m.out_col = L.REC_GATE_SILU_NORM, a.heads * a.dim
         m.max_seq = self.max_seq_len
         return m
+
+    def _layer_desc(self, d: L.MixerLayerDesc, run: int):
+        """What the driver needs beyond the mixer's block and the projections."""
+        ly = self.layers[self.runs[run]]
+        d.kind, d.norm1 = L.MIX_PARALLEL, ly.norm1.data_ptr()
+        if ly.down is not None:
+            d.norm2 = ly.norm2.data_ptr()
+
+    def _extend_model(self, x: L.MixerModelDesc, alloc):
+        """Architecture-wide parts of the driver's model description."""
 
     def _ensure_driver(self):
         if self._driver is not None:
@@ -204,17 +238,18 @@ class MixerEngine(InferenceEngine):
         cfg, R, T = self.config, self.max_rows, self.dtype
         H, P = cfg.hidden_size, min(512, self.max_seq_len)
         self.max_prefill = P
-        specs = cfg.layers
+        runs, n_runs = [self.layers[i] for i in self.runs], len(self.runs)
         alloc = self._work_allocator()
         f32 = lambda *s: alloc(s, torch.float32)
         i32 = lambda *s: alloc(s, torch.int32)
         elt = lambda *s: alloc(s, T)
-        mix = [self._mix_layer(i) for i in range(cfg.num_hidden_layers)]
+        mix = [self._mix_layer(i) for i in range(n_runs)]
+        att, rec = [m for m in mix if m.H], [m for m in mix if m.heads]
         b = self.buf = {}
         ld_x = _up8(H)
-        b["ld_proj"] = _up8(max(ly.in_proj.N for ly in self.layers))
-        b["ld_attn"] = _up8(max(ly.out_proj.K for ly in self.layers))
-        ld_act = _up8(max([ly.down.K for ly in self.layers if ly.down is not None] + [8]))
+        b["ld_proj"] = _up8(max(ly.in_proj.N for ly in runs))
+        b["ld_attn"] = _up8(max(ly.out_proj.K for ly in runs))
+        ld_act = _up8(max([ly.down.K for ly in runs if ly.down is not None] + [8]))
         b["ld_logits"] = -(-cfg.vocab_size // 4) * 4
         b["h"], b["h_tmp"], b["m"], b["xn"] = f32(R, H), f32(R, H), f32(R, H), elt(R, ld_x)
         b["proj"], b["attn_out"], b["act"] = elt(R, b["ld_proj"]), elt(R, b["ld_attn"]), elt(R, ld_act)
@@ -225,19 +260,20 @@ class MixerEngine(InferenceEngine):
         b["p_h"], b["p_m"], b["p_xn"] = f32(P, H), f32(M_PLANES, P, H), elt(P, ld_x)
         b["p_proj"], b["p_attn"], b["p_act"] = elt(P, b["ld_proj"]), elt(P, b["ld_attn"]), elt(P, ld_act)
         M = max(P, R)
-        b["qbuf"] = elt(M, max(m.H * m.dp for m in mix))
-        ld_xbc, ld_u, ld_dt = _up8(max(s.ssd.conv_channels for s in specs)), max(s.ssd.inner for s in specs), max(m.heads for m in mix)
+        b["qbuf"] = elt(M, max([m.H * m.dp for m in att] + [8]))
+        channels = [s.conv_channels for _, s in cfg.run_mixers() if s is not None]
+        ld_xbc, ld_u, ld_dt = _up8(max(channels + [8])), _up8(max([m.heads * m.P for m in rec] + [8])), max([m.heads for m in rec] + [1])
         b["xbc"], b["ubuf"], b["dtb"] = elt(M, ld_xbc), f32(M, ld_u), f32(M, ld_dt)
         # cache slices per decode-attention row: as many as the widest window can use
-        widest = max(min(m.window or self.max_seq_len, self.max_seq_len) for m in mix)
+        widest = max([min(m.window + m.keep_first if m.window else self.max_seq_len, self.max_seq_len) for m in att] + [1])
         self.attn_splits = max(1, min(32, -(-widest // 64)))
         SR = max(R, self.max_batch)                            # rows the split-attention scratch holds
-        b["attn_scratch"] = f32(max(self.lib.b2_window_attn_scratch(m.H, m.G, m.dp, SR, self.attn_splits) for m in mix))
-        b["attn_counters"] = i32(max(self.lib.b2_window_attn_units(m.H, m.G, SR) for m in mix) + 8)
-        b["ssd_counters"] = i32(max(self.lib.b2_ssd_units(C.byref(m), SR) for m in mix) + 8)
-        if self.dt == L.DT_BF16:
-            b["chunk_state"] = f32(max(self.lib.b2_ssd_chunk_state_floats(C.byref(m), P) for m in mix))
-            b["chunk_prev"] = alloc((max(self.lib.b2_ssd_chunk_prev_bytes(C.byref(m), P) for m in mix),), torch.uint8)
+        b["attn_scratch"] = f32(max([self.lib.b2_window_attn_scratch(m.H, m.G, max(m.dp, m.vp), SR, self.attn_splits) for m in att] + [8]))
+        b["attn_counters"] = i32(max([self.lib.b2_window_attn_units(m.H, m.G, SR) for m in att] + [0]) + 8)
+        b["ssd_counters"] = i32(max([self.lib.b2_ssd_units(C.byref(m), SR) for m in rec] + [0]) + 8)
+        if self.dt == L.DT_BF16 and rec:
+            b["chunk_state"] = f32(max(self.lib.b2_ssd_chunk_state_floats(C.byref(m), P) for m in rec))
+            b["chunk_prev"] = alloc((max(self.lib.b2_ssd_chunk_prev_bytes(C.byref(m), P) for m in rec),), torch.uint8)
             b["chunk_decay"] = f32(-(-P // 64) * ld_dt)
         self.argmax_blocks = max(1, min(64, cfg.vocab_size // 2048))
         b["argmax_scratch"], b["argmax_counters"] = f32(R * self.argmax_blocks * 2), i32(R + 8)
@@ -253,24 +289,25 @@ class MixerEngine(InferenceEngine):
         b["p_argmax_scratch"], b["p_argmax_counters"] = f32(self.step_rows * self.argmax_blocks * 2), i32(self.step_rows + 8)
 
         x = L.MixerModelDesc()
-        x.final_norm, x.softcap, x.dt = self.final_norm.data_ptr(), cfg.logit_softcap, self.dt
+        x.final_norm, x.softcap, x.dt = self.final_norm.data_ptr(), getattr(cfg, "logit_softcap", 0.0), self.dt
         x.ss_np, x.ld_x, x.ld_xbc, x.ld_dt, x.ld_u, x.ld_act, x.scratch_rows = self.np, ld_x, ld_xbc, ld_dt, ld_u, ld_act, SR
         x.m_planes = M_PLANES
         for k in ("m", "p_m", "qbuf", "xbc", "dtb", "ubuf", "attn_scratch", "attn_counters", "ssd_counters", "chunk_state",
                   "chunk_prev", "chunk_decay"):
             if k in b:
                 setattr(x, k, b[k].data_ptr())
-        descs = (L.MixerLayerDesc * cfg.num_hidden_layers)()
-        for i, ly in enumerate(self.layers):
-            d = descs[i]
-            d.mix, d.in_proj, d.out_proj = mix[i], ly.in_proj.desc(), ly.out_proj.desc()
-            d.norm1 = ly.norm1.data_ptr()
+        self._extend_model(x, alloc)
+        descs = (L.MixerLayerDesc * n_runs)()
+        for r, ly in enumerate(runs):
+            d = descs[r]
+            d.mix, d.in_proj, d.out_proj = mix[r], ly.in_proj.desc(), ly.out_proj.desc()
             d.gate_up.kind = d.down.kind = L.LIN_NONE
             if ly.down is not None:
-                d.gate_up, d.down, d.norm2 = ly.gate_up.desc(), ly.down.desc(), ly.norm2.data_ptr()
+                d.gate_up, d.down = ly.gate_up.desc(), ly.down.desc()
+            self._layer_desc(d, r)
         x.layers = C.addressof(descs)
         m = L.ModelDesc()
-        m.n_layers, m.H, m.vocab, m.vocab_local = cfg.num_hidden_layers, H, cfg.vocab_size, cfg.vocab_size
+        m.n_layers, m.H, m.vocab, m.vocab_local = n_runs, H, cfg.vocab_size, cfg.vocab_size
         m.max_seq, m.max_rows, m.max_prefill, m.p_logit_rows = self.max_seq_len, R, P, self.step_rows
         m.attn_splits, m.argmax_blocks, m.n_seqs_max, m.eps = self.attn_splits, self.argmax_blocks, self.max_batch, cfg.rms_norm_eps
         m.embed, m.lm_head = self.embed.data_ptr(), self.lm_head.desc()
@@ -375,5 +412,5 @@ class MixerEngine(InferenceEngine):
         from ..ops import kernels as K
         x = self._as_dev(hidden).reshape(1, -1).to(self.dtype)
         out = torch.empty(1, self.config.vocab_size, dtype=torch.float32, device=self.device)
-        K.gemv_dense(self.lm_head, x, out, mode=L.DG_STORE_F32, softcap=self.config.logit_softcap)
+        K.gemv_dense(self.lm_head, x, out, mode=L.DG_STORE_F32, softcap=getattr(self.config, "logit_softcap", 0.0))
         return out[0].cpu().numpy() if isinstance(hidden, np.ndarray) else out[0]

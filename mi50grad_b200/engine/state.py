@@ -16,7 +16,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..config import DegedraConfig, QwenConfig
+from ..config import QwenConfig
 from ..parallel.sharding import ShardSpec
 
 DN_COLS = 32
@@ -182,24 +182,25 @@ class MixerSnapshot:
 
 
 class MixerStates(SlotStates):
-    """Slots of a decoder of parallel mixers.  Every layer has arrays of its own
-    (layers may differ in size, and a layer that shares another's weights still has
-    its own history): K and V rows [slot][max_seq][kv_heads][dim padded to 8] in the
-    element type, the recurrent state [slot][heads][state][vdim] in fp32, and the
-    convolution's last taps - 1 inputs [slot][taps-1][channels]."""
+    """Slots of a decoder whose layers are described one by one.  Every run of a layer
+    has arrays of its own (layers may differ in size, and one that shares another's
+    weights, or runs several times, still has its own history): K and V rows
+    [slot][max_seq][kv_heads][dim padded to 8] in the element type, the recurrent state
+    [slot][heads][state][vdim] in fp32, and the convolution's last taps - 1 inputs
+    [slot][taps-1][channels].  What a run has not is an array of size zero."""
 
-    def __init__(self, cfg: DegedraConfig, max_seq_len: int, max_batch: int, device, dtype: torch.dtype):
+    def __init__(self, cfg, max_seq_len: int, max_batch: int, device, dtype: torch.dtype):
         super().__init__(max_batch, device)
         self.max_seq_len = max_seq_len
         z = lambda *sh, dt=dtype: torch.zeros(*sh, dtype=dt, device=device)
         self.k, self.v, self.S, self.conv = [], [], [], []
-        for l in cfg.layers:
-            a, s = l.attention, l.ssd
-            dp = -(-a.dim // 8) * 8
-            self.k.append(z(max_batch, max_seq_len, a.kv_heads, dp))
-            self.v.append(z(max_batch, max_seq_len, a.kv_heads, dp))
-            self.S.append(z(max_batch, s.heads, s.state, s.vdim, dt=torch.float32))
-            self.conv.append(z(max_batch, s.conv - 1, s.conv_channels))
+        for a, s in cfg.run_mixers():
+            G, dp, vp = (a.kv_heads, -(-a.dim // 8) * 8, -(-a.vd // 8) * 8) if a is not None else (0, 8, 8)
+            self.k.append(z(max_batch, max_seq_len, G, dp))
+            self.v.append(z(max_batch, max_seq_len, G, vp))
+            heads, N, P, taps, ch = (s.heads, s.state, s.vdim, s.conv, s.conv_channels) if s is not None else (0, 1, 1, 1, 0)
+            self.S.append(z(max_batch, heads, N, P, dt=torch.float32))
+            self.conv.append(z(max_batch, taps - 1, ch))
 
     def nbytes(self) -> int:
         return sum(t.numel() * t.element_size() for ts in (self.k, self.v, self.S, self.conv) for t in ts)

@@ -54,9 +54,25 @@ def _degedra_engine(config, device_id=0, max_seq_len=2048, **kw):
     return MixerEngine(config, device_id, max_seq_len, **kw)
 
 
+def _vekerax_config(model_dir):
+    from ..loaders.mixer import load_vekerax_config
+    return load_vekerax_config(model_dir)
+
+
+def _vekerax_loader(model_dir, config=None):
+    from ..loaders.mixer import VekeraxLoader
+    return VekeraxLoader(model_dir, config)
+
+
+def _vekerax_engine(config, device_id=0, max_seq_len=2048, **kw):
+    from ..engine.vekerax_engine import VekeraxEngine
+    return VekeraxEngine(config, device_id, max_seq_len, **kw)
+
+
 ARCHITECTURES: Dict[str, Architecture] = {
     DEFAULT: Architecture(DEFAULT, _qwen_config, _qwen_loader, _qwen_engine, ("float16",), True),
     "Degedra": Architecture("Degedra", _degedra_config, _degedra_loader, _degedra_engine, ("bfloat16", "float32"), False),
+    "Vekerax": Architecture("Vekerax", _vekerax_config, _vekerax_loader, _vekerax_engine, ("bfloat16", "float32"), False),
 }
 
 

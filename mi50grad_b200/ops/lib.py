@@ -27,7 +27,11 @@ FIN_NO_COMM, FIN_NO_H_WRITE, FIN_SAVE_EXTRA, FIN_ADD_EXTRA, FIN_NO_NORM = 1, 2, 
 FIN_TEST_WITHHOLD_SIGNAL = 32
 LIN_INT4, LIN_F16, LIN_NONE, LIN_BF16, LIN_F32 = 0, 1, 2, 3, 4
 DT_BF16, DT_F32 = 0, 1
-DG_STORE, DG_SILU_PAIR, DG_STORE_F32, DG_FMA_ROWS = 0, 1, 2, 2
+DG_STORE, DG_GATE_PAIR, DG_STORE_F32, DG_STREAMS, DG_FMA_ROWS = 0, 1, 2, 3, 2
+ACT_SILU, ACT_RELU = 0, 1
+MIX_PARALLEL, MIX_ATTENTION, MIX_RECURRENCE = 0, 1, 2
+REC_GATE_SILU_NORM, REC_NORM_SIGMOID = 0, 1
+STREAMS_MAX = 16
 STEP_EMBED_TOKENS, STEP_LM_HEAD, STEP_ARGMAX, STEP_ADVANCE, STEP_NO_COMMIT_DELTA = 1, 2, 4, 8, 16
 STEP_MATERIALIZE_XN = 32
 STEP_SPEC, STEP_GEMM_PATH, STEP_HEAD_LAST = 64, 128, 256
@@ -120,7 +124,7 @@ class GemmTcParams(C.Structure):
                 ("stages", i32), ("out", vp), ("status", vp), ("m_halves", i32), ("dense", i32),
                 ("push", vp * MAX_TP), ("epoch", vp), ("part_stride", i64), ("push_tp", i32), ("push_rank", i32),
                 ("push_per", C.c_uint), ("k_splits", i32), ("cta_pair", i32), ("bf16", i32), ("softcap", f32),
-                ("plane_stride", i64), ("box_rows", i32), ("pad3", i32)]
+                ("plane_stride", i64), ("box_rows", i32), ("act", i32), ("act_cols", i32), ("pad3", i32)]
 
 
 TC_EPI_STORE_F16, TC_EPI_SILU_PAIR, TC_EPI_STORE_F32, TC_EPI_RESID_F32 = 0, 1, 2, 3
@@ -208,25 +212,38 @@ class PostNorm(C.Structure):
     _fields_ = [("h", vp), ("m", vp), ("w", vp), ("ss", vp), ("hout", vp), ("np", i32), ("H", i32), ("eps", f32), ("pad", i32)]
 
 
+class StreamMix(C.Structure):
+    _fields_ = [("x", vp), ("u", vp), ("coef", vp), ("n", i32), ("pad", i32)]
+
+
+class StreamRows(C.Structure):
+    _fields_ = [("sm", StreamMix), ("y", vp), ("plane_stride", i64), ("planes", i32), ("pad0", i32), ("w", vp), ("xb", vp),
+                ("ldx", i32), ("rows", i32), ("H", i32), ("dt", i32), ("eps", f32), ("scale", f32),
+                ("embed", vp), ("ld_embed", i32), ("vocab", i32), ("row_tokens", vp), ("meta", vp), ("seqs", vp), ("h", vp),
+                ("from_embedding", i32), ("pad", i32)]
+
+
 class DenseGemvParams(C.Structure):
     _fields_ = [("w", vp), ("x", vp), ("pn", PostNorm), ("out", vp), ("ss_out", vp), ("ldw", i32), ("ldx", i32), ("K", i32),
                 ("N", i32), ("rows", i32), ("ldo", i32), ("mode", i32), ("dt", i32), ("rpc", i32), ("ss_np", i32),
-                ("softcap", f32), ("mma", i32)]
+                ("softcap", f32), ("mma", i32), ("act", i32), ("act_cols", i32), ("sm", StreamMix)]
 
 
 class GemmF32Params(C.Structure):
     _fields_ = [("w", vp), ("x", vp), ("out", vp), ("ldw", i32), ("ldx", i32), ("K", i32), ("N", i32), ("T", i32), ("ldo", i32),
-                ("mode", i32), ("pad", i32), ("softcap", f32), ("pad1", i32)]
+                ("mode", i32), ("act", i32), ("softcap", f32), ("act_cols", i32)]
 
 
 class MixLayer(C.Structure):
     _fields_ = [("H", i32), ("G", i32), ("d", i32), ("dp", i32), ("rot", i32), ("window", i32),
                 ("attn_scale", f32), ("left_scale", f32), ("right_scale", f32), ("eps", f32),
-                ("q_norm", vp), ("k_norm", vp), ("cos_tab", vp), ("sin_tab", vp), ("kcache", vp), ("vcache", vp),
+                ("q_norm", vp), ("k_norm", vp), ("cos_tab", vp), ("sin_tab", vp), ("kcache", vp), ("vcache", vp), ("sink", vp),
+                ("dv", i32), ("vp", i32), ("off_v", i32), ("head_norm", i32), ("keep_first", i32), ("softcap", f32),
                 ("heads", i32), ("P", i32), ("N", i32), ("groups", i32), ("ngroups", i32), ("taps", i32),
                 ("conv_w", vp), ("conv_b", vp), ("dt_bias", vp), ("A_log", vp), ("D", vp), ("norm_w", vp),
-                ("state", vp), ("conv_state", vp),
-                ("off_q", i32), ("off_k", i32), ("off_z", i32), ("off_x", i32), ("off_dt", i32), ("max_seq", i32)]
+                ("decay", vp), ("log_decay", vp), ("state", vp), ("conv_state", vp),
+                ("off_q", i32), ("off_k", i32), ("off_z", i32), ("off_x", i32), ("off_dt", i32), ("max_seq", i32),
+                ("rx", i32), ("rB", i32), ("rC", i32), ("gate", i32), ("out_col", i32), ("exact_weights", i32)]
 
 
 class MixRun(C.Structure):
@@ -239,7 +256,7 @@ class MixRun(C.Structure):
 
 class MixerLayerDesc(C.Structure):
     _fields_ = [("mix", MixLayer), ("in_proj", LinearDesc), ("out_proj", LinearDesc), ("gate_up", LinearDesc), ("down", LinearDesc),
-                ("norm1", vp), ("norm2", vp)]
+                ("norm1", vp), ("norm2", vp), ("hc1", vp), ("hc2", vp), ("kind", i32), ("act", i32), ("act_cols", i32), ("pad", i32)]
 
 
 class MixerModelDesc(C.Structure):
@@ -247,7 +264,8 @@ class MixerModelDesc(C.Structure):
                 ("ld_xbc", i32), ("ld_dt", i32), ("ld_u", i32), ("ld_act", i32), ("scratch_rows", i32), ("m_planes", i32),
                 ("m", vp), ("p_m", vp), ("qbuf", vp), ("xbc", vp), ("dtb", vp), ("ubuf", vp),
                 ("attn_scratch", vp), ("attn_counters", vp), ("ssd_counters", vp),
-                ("chunk_state", vp), ("chunk_prev", vp), ("chunk_decay", vp)]
+                ("chunk_state", vp), ("chunk_prev", vp), ("chunk_decay", vp),
+                ("streams", i32), ("ld_embed", i32), ("embed_scale", f32), ("pad", i32), ("hc0", vp), ("sx", vp), ("p_sx", vp), ("su", vp)]
 
 
 _SIZE_CHECKS = {
@@ -256,7 +274,7 @@ _SIZE_CHECKS = {
     "b2_sizeof_delta_params": DeltaParams, "b2_sizeof_argmax_params": ArgmaxParams,
     "b2_sizeof_linear_desc": LinearDesc, "b2_sizeof_layer_desc": LayerDesc,
     "b2_sizeof_model_desc": ModelDesc, "b2_sizeof_spec_stage": SpecStage, "b2_sizeof_sample_params": SampleParams, "b2_sizeof_quant8_params": Quant8Params, "b2_sizeof_act_quant_params": ActQuantParams, "b2_sizeof_gemm_tc_params": GemmTcParams, "b2_sizeof_row_meta": RowMeta, "b2_sizeof_seq_state": SeqState,
-    "b2_sizeof_dense_gemv_params": DenseGemvParams, "b2_sizeof_gemm_f32_params": GemmF32Params, "b2_sizeof_mix_layer": MixLayer,
+    "b2_sizeof_dense_gemv_params": DenseGemvParams, "b2_sizeof_gemm_f32_params": GemmF32Params, "b2_sizeof_stream_rows": StreamRows, "b2_sizeof_mix_layer": MixLayer,
     "b2_sizeof_mix_run": MixRun, "b2_sizeof_mixer_layer_desc": MixerLayerDesc, "b2_sizeof_mixer_model_desc": MixerModelDesc,
     "b2_sizeof_chain_params": ChainParams, "b2_sizeof_chain_op": ChainOp,
 }

@@ -96,7 +96,7 @@ def test_gate_up_pair(dt, F, K, rows):
     out = torch.zeros(rows, -(-F // 8) * 8, dtype=T, device="cuda")
     for rpc in (16, 32):
         out.fill_(3.0)
-        K_.gemv_dense(_lin(both, T, rpc), xs[:, :K], out, L.DG_SILU_PAIR)
+        K_.gemv_dense(_lin(both, T, rpc), xs[:, :K], out, L.DG_GATE_PAIR)
         _close(out[:, :F], ref, tol)
         assert float(out[:, F:].abs().sum()) == 0
     out.fill_(3.0)
@@ -104,7 +104,7 @@ def test_gate_up_pair(dt, F, K, rows):
     if dt == "bf16":
         K_.gemm_bf16_tc(lin.w[:, :K], xs[:, :K], out, L.TC_EPI_SILU_PAIR)
     else:
-        K_.gemm_f32(lin.w[:, :K], xs[:, :K], out, L.DG_SILU_PAIR)
+        K_.gemm_f32(lin.w[:, :K], xs[:, :K], out, L.DG_GATE_PAIR)
     _close(out[:, :F], ref, tol)
 
 
@@ -210,6 +210,7 @@ class Mix:
         m.heads, m.P, m.N, m.groups, m.ngroups, m.taps = heads, P, N, groups, ngroups, taps
         m.off_q, m.off_k, m.off_z = 0, H * d, H * d + G * d
         m.off_x, m.off_dt, m.max_seq = m.off_z + self.I, m.off_z + self.I + self.C, max_seq
+        m.dv, m.vp, m.off_v, m.rx, m.rB, m.rC, m.out_col = d, self.dp, -1, 0, self.I, self.I + groups * N, H * d
         self.ld = -(-(m.off_dt + heads) // 8) * 8
         self.ld_xbc, self.ldo = -(-self.C // 8) * 8, -(-(H * d + self.I) // 8) * 8
         lib = L.lib()
