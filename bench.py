@@ -321,10 +321,11 @@ def main():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-like-for-like", action="store_true",
                     help="skip the second timed run with fp16 attention weights (the published numbers' checkpoint layout)")
-    ap.add_argument("--mode", default="decode", choices=["decode", "batch-spec", "degedra"],
+    ap.add_argument("--mode", default="decode", choices=["decode", "batch-spec", "degedra", "vekerax"],
                     help="batch-spec: batched decode with per-step draft verification (batch x ctx, --draft tokens); "
-                         "degedra: the Degedra decoder at a few layer sizes beside the hybrid decoder of equal size")
-    ap.add_argument("--sizes", default="2k,4k,5k", help="degedra: layer sizes, with commas between them")
+                         "degedra: the Degedra decoder at a few layer sizes beside the hybrid decoder of equal size; "
+                         "vekerax: the Vekerax decoder beside Degedra of equal size")
+    ap.add_argument("--sizes", default="2k,4k,5k", help="degedra, vekerax: layer sizes, with commas between them")
     ap.add_argument("--batch", type=int, default=16)
     ap.add_argument("--ctx", type=int, default=4096)
     ap.add_argument("--draft", type=int, default=4)
@@ -354,11 +355,12 @@ def main():
     if args.impl == "torch":
         return torch_baseline(args, cfg, world, rank, local)
     from mi50grad_b200.engine.tp_engine import TPInferenceEngine
-    if args.mode == "degedra":
+    if args.mode in ("degedra", "vekerax"):
         if world != 1:
-            raise SystemExit("--mode degedra runs on one GPU")
+            raise SystemExit(f"--mode {args.mode} runs on one GPU")
         from mi50grad_b200.bench.degedra import run
-        print(json.dumps(run(args.steps, args.warmup, args.sizes.split(","), ClockSampler(local))))
+        models = {"degedra": ("degedra", "hybrid", "hybrid-fp16attn"), "vekerax": ("vekerax", "degedra")}[args.mode]
+        print(json.dumps(run(args.steps, args.warmup, args.sizes.split(","), ClockSampler(local), models)))
         return 0
     if args.mode == "batch-spec":
         return batch_spec(args, cfg, world, rank, local)

@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of the Degedra decoder at a few real layer sizes, beside the hybrid
-decoder of equal size (random weights, one GPU).  `python bench.py --mode degedra` runs all of it;
+"""Prefill and decode throughput of the dense-weight decoders at a few real layer sizes, each beside the model
+closest to it at equal size (random weights, one GPU): Degedra beside the hybrid decoder
+(`python bench.py --mode degedra`), Vekerax beside Degedra (`python bench.py --mode vekerax`).
 
-    python -m mi50grad_b200.bench.degedra --model degedra|hybrid --size 4k --phase decode|prefill --steps 2
+    python -m mi50grad_b200.bench.degedra --model vekerax|degedra|hybrid --size 4k --phase decode|prefill --steps 2
 
 runs one phase of one model a few times without timing anything (a small command for a profiler).
 """
@@ -13,7 +14,8 @@ import os
 
 import torch
 
-from ..config import DegedraConfig, EngineConfig, ParallelLayerSpec, QwenConfig, SSDSpec, WindowAttentionSpec
+from ..config import (DegedraConfig, EngineConfig, LightningSpec, ParallelLayerSpec, QwenConfig, SSDSpec, StreamLayerSpec, VekeraxConfig,
+                      WindowAttentionSpec)
 
 # width, feed-forward, attention heads / kv heads / dim, recurrence heads (of 64, state 128, 8 groups), window, layers
 SIZES = {
@@ -39,9 +41,25 @@ def hybrid_config(size: str) -> QwenConfig:
                       linear_num_key_heads=sh // 4, linear_key_head_dim=128, linear_value_head_dim=128, full_attention_interval=2)
 
 
+def vekerax_config(size: str) -> VekeraxConfig:
+    """Same width, feed-forward, layer count and vocabulary; attention and lightning layers in turn, each mixer as
+    wide as its counterpart in the Degedra layer (recurrent state of the same size in heads of 128), four streams."""
+    w, ff, h, kv, d, sh, win, n = SIZES[size]
+    att = StreamLayerSpec(WindowAttentionSpec(h, kv, d, 0, 0.0, d ** -0.5, win, vdim=d, head_norm=True, keep_first=4, softcap=30.0, sink=True), ff)
+    rec = StreamLayerSpec(LightningSpec(sh // 2, 128, 128, tuple(1.0 - 2.0 ** (-1 - 8 * i / sh) for i in range(sh // 2))), ff)
+    return VekeraxConfig(w, VOCAB, 1e-5, [att if i % 2 == 0 else rec for i in range(n)], 1.0, 1.0, 4)
+
+
+MODELS = ("vekerax", "degedra", "hybrid", "hybrid-fp16attn")
+
+
 def make(model: str, size: str, max_seq: int, batch: int):
     ecfg = EngineConfig(max_step_rows=64)
-    if model == "degedra":
+    if model == "vekerax":
+        from ..engine.vekerax_engine import VekeraxEngine
+        eng = VekeraxEngine(vekerax_config(size), max_seq_len=max_seq, max_batch=batch, engine_config=ecfg)
+        eng.init_random(0)
+    elif model == "degedra":
         from ..engine.mixer_engine import MixerEngine
         eng = MixerEngine(degedra_config(size), max_seq_len=max_seq, max_batch=batch, engine_config=ecfg)
         eng.init_random(0)
@@ -117,7 +135,8 @@ def measure(model: str, size: str, steps: int, warmup: int, peaks: dict) -> dict
     return out
 
 
-def run(steps: int, warmup: int, sizes, sampler) -> dict:
+def run(steps: int, warmup: int, sizes, sampler, models=("degedra", "hybrid", "hybrid-fp16attn")) -> dict:
+    """models[0] is the one the headline value is of; the others stand beside it."""
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
     path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
     if os.path.exists(path):
@@ -126,17 +145,19 @@ def run(steps: int, warmup: int, sizes, sampler) -> dict:
     sampler.start()
     for size in sizes:
         res[size] = {}
-        for model in ("degedra", "hybrid", "hybrid-fp16attn"):
+        for model in models:
             res[size][model] = measure(model, size, steps, warmup, peaks)
             torch.cuda.empty_cache()
     clocks = sampler.stop()
-    first = sizes[-1]
+    first, main_model = sizes[-1], models[0]
+    name = main_model.capitalize()
+    dtype = "bf16 (hybrid: int4 weights, fp16 activations)" if "hybrid" in models else "bf16"
     return {
-        "metric": f"decode tok/s (bs1), Degedra {first} layers", "value": res[first]["degedra"]["decode_bs1_tok_s"], "unit": "tok/s",
-        "n_gpus": 1, "steps": steps, "warmup": max(3, warmup), "ms_per_step": res[first]["degedra"]["decode_bs1_ms"],
-        "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16 (hybrid: int4 weights, fp16 activations)",
+        "metric": f"decode tok/s (bs1), {name} {first} layers", "value": res[first][main_model]["decode_bs1_tok_s"], "unit": "tok/s",
+        "n_gpus": 1, "steps": steps, "warmup": max(3, warmup), "ms_per_step": res[first][main_model]["decode_bs1_ms"],
+        "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": dtype,
         "data": "synthetic (random weights and token ids)", "impl": "ours", "clocks": clocks, "peaks": peaks,
-        "config": {"model": "Degedra", "global_batch": 1, "seq_len": 512, "parallelism": "tp1", "vocab": VOCAB,
+        "config": {"model": name, "global_batch": 1, "seq_len": 512, "parallelism": "tp1", "vocab": VOCAB,
                    "sizes": {k: dict(zip(("width", "ff", "heads", "kv_heads", "dim", "ssd_heads", "window", "layers"), SIZES[k])) for k in sizes},
                    "l2": "inputs larger than L2 (weights of all layers per step)"},
         "results": res,
@@ -145,7 +166,7 @@ def run(steps: int, warmup: int, sizes, sampler) -> dict:
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="degedra", choices=["degedra", "hybrid", "hybrid-fp16attn"])
+    ap.add_argument("--model", default="degedra", choices=MODELS)
     ap.add_argument("--size", default="4k", choices=sorted(SIZES))
     ap.add_argument("--phase", default="decode", choices=["decode", "prefill"])
     ap.add_argument("--steps", type=int, default=2)

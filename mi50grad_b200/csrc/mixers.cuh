@@ -95,7 +95,7 @@ __device__ __forceinline__ void stream_mix(int n, float* x, const float* coef, i
         case 3: stream_mix_n<3, W>(x, coef, H, y); return;
         case 4: stream_mix_n<4, W>(x, coef, H, y); return;
     }
-#pragma unroll 1
+#pragma unroll
     for (int e = 0; e < W; ++e) {
         float v[STREAMS_MAX], u = 0.f;
 #pragma unroll 1

@@ -194,6 +194,12 @@ static bool ssd_valid(const MixLayer* l) {
            l->ngroups >= 1 && (l->heads * l->P) % l->ngroups == 0 && l->taps >= 1 && (l->decay ? l->log_decay != nullptr : l->A_log != nullptr);
 }
 
+// one CTA per part of a row, with a thread for every four columns of it
+template <typename T>
+static int launch_ssd_norm(const MixLayer* l, const MixRun* r, cudaStream_t s) {
+    const int w4 = (l->heads * l->P / l->ngroups + 3) / 4, nt = w4 >= 256 ? 256 : (w4 + 31) / 32 * 32;
+    return launch_pdl(ssd_norm_kernel<T>, dim3(r->n_rows, l->ngroups), dim3(nt), 0, s, *l, *r);
+}
 template <typename T>
 static int launch_ssd_step(const MixLayer* l, const MixRun* r, cudaStream_t s) {
     dim3 grid(l->heads, (l->P + 31) / 32, r->n_seqs);
@@ -202,7 +208,7 @@ static int launch_ssd_step(const MixLayer* l, const MixRun* r, cudaStream_t s) {
     else if (l->N <= 128) e = launch_pdl(ssd_step_kernel<T, 16>, grid, dim3(SS_THREADS), 0, s, *l, *r);
     else e = launch_pdl(ssd_step_kernel<T, 32>, grid, dim3(SS_THREADS), 0, s, *l, *r);
     if (e || r->fuse_norm) return e;
-    return launch_pdl(ssd_norm_kernel<T>, dim3(r->n_rows, l->ngroups), dim3(256), 0, s, *l, *r);
+    return launch_ssd_norm<T>(l, r, s);
 }
 // Any mix of sequences; fuse_norm = 0 adds a launch for the norm (many rows per sequence).
 B2_API int b2_ssd_step(const MixLayer* l, const MixRun* r, cudaStream_t s) {
@@ -488,7 +494,7 @@ B2_API int b2_ssd_chunk(const MixLayer* l, const MixRun* r, cudaStream_t s) {
     if (int e = launch_pdl(ssd_chunk_state_kernel, dim3(chunks, l->heads, pb), dim3(128), sm1, s, *l, *r)) return e;
     if (int e = launch_pdl(ssd_chunk_pass_kernel, dim3((l->N * Pp + 255) / 256, l->heads), dim3(256), 0, s, *l, *r, chunks)) return e;
     if (int e = launch_pdl(ssd_chunk_out_kernel, dim3(chunks, l->heads, pb), dim3(128), sm3, s, *l, *r)) return e;
-    return launch_pdl(ssd_norm_kernel<bf16>, dim3(r->n_rows, l->ngroups), dim3(256), 0, s, *l, *r);
+    return launch_ssd_norm<bf16>(l, r, s);
 }
 B2_API long long b2_ssd_chunk_state_floats(const MixLayer* l, int rows) {
     return (long long)((rows + SC_T - 1) / SC_T) * l->heads * l->N * l->P;

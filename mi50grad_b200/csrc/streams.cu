@@ -5,8 +5,6 @@
 // the last one the input weights are all one and the norm is the final norm.  The streams are fp32.
 #include "mixers.cuh"
 
-#define SR_THREADS 256
-
 template <typename T>
 __device__ __forceinline__ void store4(T* d, const float (&o)[4]) {
     if constexpr (sizeof(T) == 2) {
@@ -27,13 +25,13 @@ __device__ __forceinline__ void load_e(const T* p, float (&v)[W]) {
         for (int e = 0; e < W; ++e) v[e] = ld_f(p + e);
 }
 
-// W = 4 (PER > 0): H % 4 == 0, at most PER * 1024 columns, and a row's u stays in registers between the passes
-template <typename T, int W, int PER>
-__global__ void __launch_bounds__(SR_THREADS) stream_rows_kernel(const StreamRows p) {
+// W = 4 (PER > 0): H % 4 == 0, at most PER * NT * 4 columns, and a row's u stays in registers between the passes
+template <typename T, int W, int PER, int NT>
+__global__ void __launch_bounds__(NT) stream_rows_kernel(const StreamRows p) {
     __shared__ float red[32], coef[STREAMS_MAX * (STREAMS_MAX + 2)];
     pdl_launch_dependents();
     const int r = blockIdx.x, tid = threadIdx.x, n = p.sm.n, H = p.H;
-    for (int i = tid; i < n * (n + 2); i += SR_THREADS) coef[i] = p.sm.coef[i];
+    for (int i = tid; i < n * (n + 2); i += NT) coef[i] = p.sm.coef[i];
     __syncthreads();
     pdl_wait();
     float* x = p.sm.x + (size_t)r * n * H;
@@ -82,7 +80,7 @@ __global__ void __launch_bounds__(SR_THREADS) stream_rows_kernel(const StreamRow
         float u[PER][4];
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int c = (tid + k * SR_THREADS) * 4;
+            const int c = (tid + k * NT) * 4;
 #pragma unroll
             for (int e = 0; e < 4; ++e) u[k][e] = 0.f;
             if (c < H) column(c, u[k]);
@@ -92,7 +90,7 @@ __global__ void __launch_bounds__(SR_THREADS) stream_rows_kernel(const StreamRow
         const float inv = rsqrtf(block_sum(ss, red) / (float)H + p.eps);
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int c = (tid + k * SR_THREADS) * 4;
+            const int c = (tid + k * NT) * 4;
             if (c >= H) continue;
             float w[4];
             load_e<float, 4>(p.w + c, w);
@@ -101,13 +99,13 @@ __global__ void __launch_bounds__(SR_THREADS) stream_rows_kernel(const StreamRow
             store4<T>(xb + c, w);
         }
     } else {
-        for (int c = tid; c < H; c += SR_THREADS) {
+        for (int c = tid; c < H; c += NT) {
             float u[1];
             column(c, u);
             ss += u[0] * u[0];
         }
         const float inv = rsqrtf(block_sum(ss, red) / (float)H + p.eps);
-        for (int c = tid; c < H; c += SR_THREADS) {              // (a thread re-reads only what it wrote)
+        for (int c = tid; c < H; c += NT) {              // (a thread re-reads only what it wrote)
             float v = 0.f;
             for (int s = 0; s < n; ++s) v = fmaf(coef[n * n + n + s], x[(size_t)s * H + c], v);
             xb[c] = to_t<T>(v * inv * p.w[c]);
@@ -118,17 +116,20 @@ __global__ void __launch_bounds__(SR_THREADS) stream_rows_kernel(const StreamRow
 template <typename T>
 static int launch_sr(const StreamRows* p, cudaStream_t s) {
     const bool vec = (p->H & 3) == 0 && p->H <= 8192 && (p->ldx & 3) == 0 && (p->plane_stride & 3) == 0 && (p->ld_embed & 3) == 0;
-    const dim3 g(p->rows), b(SR_THREADS);
-    auto go = [&](auto kern) -> int {
+    auto go = [&](auto kern, int threads) -> int {
+        const dim3 g(p->rows), b(threads);
         // the embedding is a plain launch: whatever follows in the step may rely on prepare_rows (which precedes it) being complete
         if (p->from_embedding) { kern<<<g, b, 0, s>>>(*p); return cudaGetLastError(); }
         return launch_pdl(kern, g, b, 0, s, *p);
     };
-    if (!vec) return go(stream_rows_kernel<T, 1, 0>);
-    if (p->H <= 1024) return go(stream_rows_kernel<T, 4, 1>);
-    if (p->H <= 2048) return go(stream_rows_kernel<T, 4, 2>);
-    if (p->H <= 4096) return go(stream_rows_kernel<T, 4, 4>);
-    return go(stream_rows_kernel<T, 4, 8>);
+    if (!vec) return go(stream_rows_kernel<T, 1, 0, 256>, 256);
+    // A thread's groups of four columns go one after another, so few per thread are fast as long as the CTAs that
+    // leaves on an SM still cover each other's barriers: 1024 threads up to 64 rows, 512 beyond.  (512 rows of 4096
+    // columns, four streams: 17.3 us, with 256 threads 22.0; one row 3.8, 4.4 and 6.0.)
+    const int nt = p->rows <= 64 ? 1024 : 512, per = (p->H + 4 * nt - 1) / (4 * nt);
+    if (nt == 1024) return per <= 1 ? go(stream_rows_kernel<T, 4, 1, 1024>, 1024) : go(stream_rows_kernel<T, 4, 2, 1024>, 1024);
+    if (per <= 1) return go(stream_rows_kernel<T, 4, 1, 512>, 512);
+    return per <= 2 ? go(stream_rows_kernel<T, 4, 2, 512>, 512) : go(stream_rows_kernel<T, 4, 4, 512>, 512);
 }
 B2_API int b2_stream_rows(const StreamRows* p, cudaStream_t s) {
     if (p->rows < 1 || p->H < 1 || p->sm.n < 1 || p->sm.n > STREAMS_MAX || !p->sm.x || !p->sm.coef || !p->w || !p->xb || p->ldx < p->H ||

@@ -515,7 +515,7 @@ def wait_self_test(wait_us: int = 2000) -> dict:
 
 
 # ---------------------------------------------------------------------------
-# Dense-weight, post-norm decoder path (csrc/mixers.cuh)
+# Dense-weight decoder path (csrc/mixers.cuh)
 # ---------------------------------------------------------------------------
 
 def _dt(t: torch.Tensor) -> int:
@@ -532,10 +532,27 @@ def post_norm_input(h: torch.Tensor, m: Optional[torch.Tensor] = None, w: Option
     return pn
 
 
+def norm_input(u: torch.Tensor, w: torch.Tensor, ss: torch.Tensor, eps: float = 1e-6) -> L.PostNorm:
+    """Input descriptor of `gemv_dense`: x = u * rsqrt(sum(ss[row]) / H + eps) * w."""
+    pn = post_norm_input(u, u, w, ss, None, eps)
+    pn.h = None
+    return pn
+
+
+def stream_mix(x: torch.Tensor, u: Optional[torch.Tensor], coef: torch.Tensor) -> L.StreamMix:
+    """Residual streams x [rows, n, H] (updated in place), u [rows, H], coef = mix [n, n] | out [n] | in [n]."""
+    sm = L.StreamMix()
+    sm.x, sm.u, sm.coef, sm.n = x.data_ptr(), L.ptr(u), coef.data_ptr(), x.shape[1]
+    sm.tensors = (x, u, coef)
+    return sm
+
+
 def gemv_dense(lin, x: Optional[torch.Tensor], out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0,
-               pn: Optional[L.PostNorm] = None, rows: Optional[int] = None, ss_out: Optional[torch.Tensor] = None, mma: bool = False):
+               pn: Optional[L.PostNorm] = None, rows: Optional[int] = None, ss_out: Optional[torch.Tensor] = None, mma: bool = False, act: int = L.ACT_SILU,
+               act_cols: int = 0, sm: Optional[L.StreamMix] = None):
     """1..8 rows times a `MixerLinear`-like object (.w [N][ldw], .K, .N, .rpc_few, .rpc); bf16 or fp32.
-    mma: the tensor-core kernel also for one or two bf16 rows."""
+    mma: the tensor-core kernel also for one or two bf16 rows.  DG_GATE_PAIR: act(gate) * up; DG_STORE: SiLU on the
+    first act_cols outputs; DG_STREAMS: the product goes into the streams `sm` (out is None)."""
     p = L.DenseGemvParams()
     n = rows if x is None else x.shape[0]
     tc = lin.w.dtype == torch.bfloat16 and (mma or n > L.DG_FMA_ROWS)
@@ -545,18 +562,24 @@ def gemv_dense(lin, x: Optional[torch.Tensor], out: torch.Tensor, mode: int = L.
         p.x, p.ldx, p.rows = x.data_ptr(), x.stride(0), x.shape[0]
     else:
         p.pn, p.rows = pn, rows
-    p.out, p.ldo, p.mode, p.softcap = out.data_ptr(), out.stride(0), mode, softcap
+    p.mode, p.softcap, p.act, p.act_cols = mode, softcap, act, act_cols
+    if sm is not None:
+        p.sm = sm
+    else:
+        p.out, p.ldo = out.data_ptr(), out.stride(0)
     if ss_out is not None:
         p.ss_out, p.ss_np = ss_out.data_ptr(), ss_out.shape[1]
     L.check(L.lib().b2_gemv_dense(C.byref(p), L.stream()), "gemv_dense")
     return out
 
 
-def gemm_f32(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0):
+def gemm_f32(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, mode: int = L.DG_STORE, softcap: float = 0.0,
+             act: int = L.ACT_SILU, act_cols: int = 0):
     """out[t][n] = x[t] . w[n] in true fp32."""
     p = L.GemmF32Params()
     p.w, p.x, p.out, p.ldw, p.ldx, p.ldo = w.data_ptr(), x.data_ptr(), out.data_ptr(), w.stride(0), x.stride(0), out.stride(0)
     p.K, p.N, p.T, p.mode, p.softcap = x.shape[1], w.shape[0], x.shape[0], mode, softcap
+    p.act, p.act_cols = act, act_cols
     L.check(L.lib().b2_gemm_f32(C.byref(p), L.stream()), "gemm_f32")
     return out
 
@@ -573,7 +596,8 @@ def post_norm_(h: torch.Tensor, m: Optional[torch.Tensor], w: Optional[torch.Ten
 
 
 def gemm_bf16_tc(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, epi: int = L.TC_EPI_STORE_F32,
-                 t_tile: Optional[int] = None, softcap: float = 0.0, cta_pair: bool = False, k_splits: int = 1):
+                 t_tile: Optional[int] = None, softcap: float = 0.0, cta_pair: bool = False, k_splits: int = 1,
+                 act: int = L.ACT_SILU, act_cols: int = 0):
     """out[t][n] (epi) = x[t] . w[n] for bf16 operands on the tcgen05 tensor cores; any K (row strides
     multiples of 8).  k_splits > 1: out is [planes][T][N] fp32, the product is the sum of its planes."""
     T, dev = x.shape[0], x.device
@@ -584,12 +608,36 @@ def gemm_bf16_tc(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, epi: int =
     p.K, p.T, p.t_tile, p.epi = x.shape[1], T, t_tile or min(256, -(-T // 16) * 16), epi
     p.n_valid = w.shape[0] // 2 if epi == L.TC_EPI_SILU_PAIR else w.shape[0]
     p.ldo, p.out, p.status, p.bf16, p.softcap = out.stride(-2), out.data_ptr(), st.data_ptr(), 1, softcap
+    p.act, p.act_cols = act, act_cols
     p.cta_pair, p.k_splits, p.plane_stride = int(cta_pair), k_splits, out.stride(0) if out.dim() == 3 else 0
     L.check(L.lib().b2_gemm_f16_tc(C.byref(p), C.c_void_p(w.data_ptr()), w.stride(0), C.c_void_p(x.data_ptr()),
                                    x.stride(0), L.stream()), "gemm_bf16_tc")
     return out
 
 
+def stream_rows(x: torch.Tensor, coef: torch.Tensor, w: torch.Tensor, xb: torch.Tensor, eps: float, y: Optional[torch.Tensor] = None,
+                u: Optional[torch.Tensor] = None, h: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None,
+                tokens: Optional[torch.Tensor] = None, rows_meta: Optional[torch.Tensor] = None, seqs: Optional[torch.Tensor] = None,
+                scale: float = 1.0):
+    """Streams x [rows, n, H] take the sublayer output y [rows, H] (or planes [p, rows, H]); xb = the norm of the next
+    sublayer's input, u (optional) that input.  Without y the streams are filled with scale times the rows `h`, or
+    the rows of `embed` that `tokens` (a token < 0: the sequence's own) choose."""
+    p = L.StreamRows()
+    p.sm = stream_mix(x, u, coef)
+    p.rows, p.H, p.w, p.xb, p.ldx = x.shape[0], x.shape[2], w.data_ptr(), xb.data_ptr(), xb.stride(0)
+    p.dt, p.eps, p.scale, p.planes = _dt(xb), eps, scale, 1
+    if y is not None:
+        p.y = y.data_ptr()
+        if y.dim() == 3:
+            p.planes, p.plane_stride = y.shape[0], y.stride(0)
+    else:
+        p.from_embedding, p.h = 1, L.ptr(h)
+        if embed is not None:
+            p.embed, p.ld_embed, p.vocab = embed.data_ptr(), embed.stride(0), embed.shape[0]
+            p.row_tokens, p.meta, p.seqs = L.ptr(tokens), rows_meta.data_ptr(), seqs.data_ptr()
+    L.check(L.lib().b2_stream_rows(C.byref(p), L.stream()), "stream_rows")
+
+
 def mix_op(name: str, layer: L.MixLayer, run: L.MixRun):
-    """Launch one mixer kernel: 'mix_prepare', 'window_attn_decode', 'window_attn_rows', 'ssd_step', 'ssd_chunk'."""
+    """Launch one mixer kernel: 'mix_prepare', 'head_prepare', 'window_attn_decode', 'window_attn_rows', 'ssd_step', 'ssd_chunk'."""
     L.check(getattr(L.lib(), "b2_" + name)(C.byref(layer), C.byref(run), L.stream()), name)

@@ -34,3 +34,15 @@ def test_degedra_mode_compares_models_of_equal_size():
         assert (d.hidden_size, l.ff, len(d.layers), d.vocab_size) == (h.hidden_size, h.intermediate_size, h.num_hidden_layers, h.vocab_size)
         assert l.attention.heads * l.attention.dim == h.full_attn_q_dim
         assert l.ssd.inner == h.linear_attn_value_dim
+
+
+def test_vekerax_mode_compares_models_of_equal_size():
+    src = open(os.path.join(ROOT, "bench.py")).read()
+    assert '"vekerax": ("vekerax", "degedra")' in src
+    from mi50grad_b200.bench.degedra import SIZES, degedra_config, vekerax_config
+    for size in SIZES:
+        v, d = vekerax_config(size), degedra_config(size)
+        assert (v.hidden_size, v.vocab_size, len(v.layers), v.layers[0].ff) == (d.hidden_size, d.vocab_size, len(d.layers), d.layers[0].ff)
+        a, r, l = v.layers[0].attention, v.layers[1].recurrence, d.layers[0]
+        assert (a.heads, a.kv_heads, a.dim, a.vd, a.window) == (l.attention.heads, l.attention.kv_heads, l.attention.dim, l.attention.vd, l.attention.window)
+        assert r.heads * r.state * r.vdim == l.ssd.heads * l.ssd.state * l.ssd.vdim and r.inner == l.ssd.inner
