@@ -253,16 +253,26 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                 uint32_t r[32];
                 tc_ld32(tmem_base + ((uint32_t)(lg * 32) << 16) + (uint32_t)(hc * 256 + c0), r);
                 tc_wait_ld();
+                // (one unrolled loop per form: a warp then walks only its own form's instructions)
                 if (p.epi == TC_EPI_SILU_PAIR) {
                     const bool is_gate = (lane & 8) == 0;
                     const int o = blockIdx.x * (TC_BM / 2 * MH) + hc * (TC_BM / 2) + lg * 16 + (lane >> 4) * 8 + (lane & 7);
+                    if (p.act) {
+#pragma unroll
+                        for (int c = 0; c < 32; ++c) {
+                            const float v = __uint_as_float(r[c]), up = __shfl_down_sync(0xffffffffu, v, 8);
+                            const int tt = t0 + c0 + c;
+                            if (is_gate && c0 + c < Tp && tt < p.T && o < p.n_valid) tc_store16(p, (size_t)tt * p.ldo + o, fmaxf(v, 0.f) * up);
+                        }
+                        continue;
+                    }
 #pragma unroll
                     for (int c = 0; c < 32; ++c) {
                         float v = __uint_as_float(r[c]);
                         float up = __shfl_down_sync(0xffffffffu, v, 8);
                         int tt = t0 + c0 + c;
                         if (is_gate && c0 + c < Tp && tt < p.T && o < p.n_valid)
-                            tc_store16(p, (size_t)tt * p.ldo + o, (p.act ? fmaxf(v, 0.f) : silu_f(v)) * up);
+                            tc_store16(p, (size_t)tt * p.ldo + o, silu_f(v) * up);
                     }
                 } else if (p.epi == TC_EPI_PUSH_F32) {
                     // plain stores into the owner's memory over NVLink (posted writes, 128 bytes per warp)
@@ -277,17 +287,34 @@ gemm_int4_tc_kernel(const GemmTcParams p, const __grid_constant__ CUtensorMap xm
                             *dst = __uint_as_float(r[c]);
                         }
                     }
+                } else if (p.epi == TC_EPI_STORE_F16) {
+                    if (n < p.act_cols) {
+#pragma unroll
+                        for (int c = 0; c < 32; ++c) r[c] = __float_as_uint(silu_f(__uint_as_float(r[c])));
+                    }
+#pragma unroll
+                    for (int c = 0; c < 32; ++c) {
+                        const int tt = t0 + c0 + c;
+                        if (c0 + c < Tp && tt < p.T && n < p.n_valid) tc_store16(p, (size_t)tt * p.ldo + n, __uint_as_float(r[c]));
+                    }
+                } else if (p.epi == TC_EPI_STORE_F32) {
+                    if (p.softcap > 0.f) {
+#pragma unroll
+                        for (int c = 0; c < 32; ++c) r[c] = __float_as_uint(p.softcap * tanhf(__uint_as_float(r[c]) / p.softcap));
+                    }
+#pragma unroll
+                    for (int c = 0; c < 32; ++c) {
+                        const int tt = t0 + c0 + c;
+                        if (c0 + c < Tp && tt < p.T && n < p.n_valid) ((float*)p.out)[(size_t)tt * p.ldo + n + plane] = __uint_as_float(r[c]);
+                    }
                 } else {
 #pragma unroll
                     for (int c = 0; c < 32; ++c) {
-                        int tt = t0 + c0 + c;
+                        const int tt = t0 + c0 + c;
                         if (c0 + c < Tp && tt < p.T && n < p.n_valid) {
-                            float v = __uint_as_float(r[c]);
-                            size_t o = (size_t)tt * p.ldo + n;
-                            if (p.epi == TC_EPI_STORE_F16) tc_store16(p, o, n < p.act_cols ? silu_f(v) : v);
-                            else if (p.epi == TC_EPI_STORE_F32) ((float*)p.out)[o + plane] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
-                            else if (gridDim.z > 1) atomicAdd((float*)p.out + o, v);     // split-K partial
-                            else ((float*)p.out)[o] += v;
+                            float* o = (float*)p.out + (size_t)tt * p.ldo + n;
+                            if (gridDim.z > 1) atomicAdd(o, __uint_as_float(r[c]));     // split-K partial
+                            else *o += __uint_as_float(r[c]);
                         }
                     }
                 }

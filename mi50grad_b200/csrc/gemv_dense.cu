@@ -55,12 +55,13 @@ __device__ __forceinline__ void pn_inverse(const PostNorm& n, int rows, float* i
     s = warp_sum(s);
     if (lane == 0) inv[warp] = rsqrtf(s / (float)n.H + n.eps);
 }
-// Four columns [k, k + 4) of row m of the updated stream; CTA (k / 4) mod gridDim stores them.
+// Four columns [k, k + 4) of row m of the updated stream; CTA (k / 4) mod gridDim stores them.  (EXT: see dg_extended)
+template <bool EXT>
 __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const float* inv, float (&v)[4]) {
     const size_t o = (size_t)m * n.H + k;
     const bool mine = (k >> 2) % (int)gridDim.x == (int)blockIdx.x;
     if ((n.H & 3) == 0) {
-        if (!n.h) {
+        if (EXT && !n.h) {
             const float4 m4 = *(const float4*)(n.m + o), w4 = *(const float4*)(n.w + k);
             const float iv = inv[m];
             v[0] = m4.x * iv * w4.x; v[1] = m4.y * iv * w4.y; v[2] = m4.z * iv * w4.z; v[3] = m4.w * iv * w4.w;
@@ -79,7 +80,7 @@ __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const 
         for (int e = 0; e < 4; ++e) {
             v[e] = 0.f;
             if (k + e < n.H) {
-                if (!n.h) { v[e] = n.m[o + e] * inv[m] * n.w[k + e]; continue; }
+                if (EXT && !n.h) { v[e] = n.m[o + e] * inv[m] * n.w[k + e]; continue; }
                 v[e] = n.h[o + e];
                 if (n.m) { v[e] += n.m[o + e] * inv[m] * n.w[k + e]; if (mine) n.hout[o + e] = v[e]; }
             }
@@ -87,8 +88,12 @@ __device__ __forceinline__ void pn_load4(const PostNorm& n, int m, int k, const 
     }
 }
 
+// Launches that need what only decoders over residual streams use (the plain norm of the input, the update of the
+// streams, activations other than the SiLU pair) run instantiations of their own, so that the others stay lean.
+static bool dg_extended(const DenseGemvParams& p) { return p.mode == DG_STREAMS || p.act || p.act_cols > 0 || (!p.x && !p.pn.h); }
+
 // Finished [rpc][8] tile in y_s -> output (both element types).
-template <typename T>
+template <typename T, bool EXT>
 __device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, float (*y_s)[8], int tid, int lane, int warp) {
     const int n0 = blockIdx.x * p.rpc;
     if (p.mode == DG_GATE_PAIR) {
@@ -96,7 +101,7 @@ __device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, float (*y_
         for (int i = tid; i < half * p.rows; i += DG_THREADS) {
             const int m = i / half, j = i % half, nl = (j >> 3) * 16 + (j & 7), o = blockIdx.x * half + j;
             const float g = y_s[nl][m];
-            if (2 * o < p.N) ((T*)p.out)[(size_t)m * p.ldo + o] = to_t<T>((p.act == ACT_RELU ? fmaxf(g, 0.f) : silu_p(g)) * y_s[nl + 8][m]);
+            if (2 * o < p.N) ((T*)p.out)[(size_t)m * p.ldo + o] = to_t<T>((EXT && p.act == ACT_RELU ? fmaxf(g, 0.f) : silu_p(g)) * y_s[nl + 8][m]);
         }
         return;
     }
@@ -104,15 +109,15 @@ __device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, float (*y_
         const int m = i / p.rpc, nl = i % p.rpc, n = n0 + nl;
         if (n >= p.N) continue;
         const float v = y_s[nl][m];
-        if (p.mode == DG_STORE) ((T*)p.out)[(size_t)m * p.ldo + n] = to_t<T>(n < p.act_cols ? silu_p(v) : v);
-        else if (p.mode == DG_STREAMS) {
+        if (p.mode == DG_STORE) ((T*)p.out)[(size_t)m * p.ldo + n] = to_t<T>(EXT && n < p.act_cols ? silu_p(v) : v);
+        else if (EXT && p.mode == DG_STREAMS) {
             float y[1] = {v};
             stream_mix<1>(p.sm.n, p.sm.x + (size_t)m * p.sm.n * p.N + n, p.sm.coef, p.N, y);
             p.sm.u[(size_t)m * p.N + n] = y_s[nl][m] = y[0];
         } else ((float*)p.out)[(size_t)m * p.ldo + n] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
     }
-    if (p.mode == DG_STREAMS) __syncthreads();
-    if (p.mode >= DG_STORE_F32 && p.ss_out && warp < p.rows) {
+    if (EXT && p.mode == DG_STREAMS) __syncthreads();
+    if ((p.mode == DG_STORE_F32 || (EXT && p.mode == DG_STREAMS)) && p.ss_out && warp < p.rows) {
         float s = 0.f;
         for (int nl = lane; nl < p.rpc; nl += 32) if (n0 + nl < p.N) s += y_s[nl][warp] * y_s[nl][warp];
         s = warp_sum(s);
@@ -120,6 +125,7 @@ __device__ __forceinline__ void dg_epilogue(const DenseGemvParams& p, float (*y_
     }
 }
 
+template <bool EXT>
 __global__ void __launch_bounds__(DG_THREADS, 2) gemv_bf16_kernel(const DenseGemvParams p, int KC) {
     extern __shared__ __align__(16) unsigned char dg_smem[];
     bf16* xs = (bf16*)dg_smem;                              // [1 or 2][rows][KC + DM_PAD]
@@ -168,7 +174,7 @@ __global__ void __launch_bounds__(DG_THREADS, 2) gemv_bf16_kernel(const DenseGem
         for (int i = tid * 4; i < p.rows * kl; i += DG_THREADS * 4) {
             const int m = i / kl, k = i % kl;
             float v[4] = {0.f, 0.f, 0.f, 0.f};
-            if (k < p.K) pn_load4(p.pn, m, k, inv_s, v);
+            if (k < p.K) pn_load4<EXT>(p.pn, m, k, inv_s, v);
             uint2 pk; pk.x = dm_pack(v[0], v[1]); pk.y = dm_pack(v[2], v[3]);
             *(uint2*)(xs + (size_t)m * LDX + k) = pk;
         }
@@ -208,9 +214,10 @@ __global__ void __launch_bounds__(DG_THREADS, 2) gemv_bf16_kernel(const DenseGem
         y_s[nl][m] = v;
     }
     __syncthreads();
-    dg_epilogue<bf16>(p, y_s, tid, lane, warp);
+    dg_epilogue<bf16, EXT>(p, y_s, tid, lane, warp);
 }
 
+template <bool EXT>
 static int launch_dm(const DenseGemvParams* p, cudaStream_t s) {
     const int WK = DG_WARPS / (p->rpc >> 4), unit = 64 * WK * DM_D, Kr = (p->K + unit - 1) / unit * unit;
     int KC = Kr;
@@ -225,8 +232,8 @@ static int launch_dm(const DenseGemvParams* p, cudaStream_t s) {
     const size_t smem = (size_t)(two ? 2 : 1) * p->rows * (KC + DM_PAD) * 2;
     if (smem > 200 << 10) return cudaErrorInvalidValue;     // (a PostNorm input wider than shared memory)
     static SmemOptIn opt;
-    if (int e = opt.ensure((const void*)gemv_bf16_kernel, smem)) return e;
-    return launch_pdl(gemv_bf16_kernel, dim3((p->N + p->rpc - 1) / p->rpc), dim3(DG_THREADS), smem, s, *p, KC);
+    if (int e = opt.ensure((const void*)gemv_bf16_kernel<EXT>, smem)) return e;
+    return launch_pdl(gemv_bf16_kernel<EXT>, dim3((p->N + p->rpc - 1) / p->rpc), dim3(DG_THREADS), smem, s, *p, KC);
 }
 
 // ---------------------------------------------------------------------------
@@ -248,7 +255,7 @@ template <> struct DgVec<float> {
     }
 };
 
-template <typename T, int MR>
+template <typename T, int MR, bool EXT>
 __global__ void __launch_bounds__(DG_THREADS) gemv_fma_kernel(const DenseGemvParams p, int KC) {
     constexpr int V = DgVec<T>::V;
     extern __shared__ __align__(16) unsigned char dg_smem[];
@@ -301,7 +308,7 @@ __global__ void __launch_bounds__(DG_THREADS) gemv_fma_kernel(const DenseGemvPar
                 const int m = i / KC, kk = i % KC, kg = c0 + kk;
                 if (kk >= cl) continue;
                 float v[4] = {0.f, 0.f, 0.f, 0.f};
-                if (!p.x) { if (kg < p.K) pn_load4(p.pn, m, kg, inv_s, v); }
+                if (!p.x) { if (kg < p.K) pn_load4<EXT>(p.pn, m, kg, inv_s, v); }
                 else
 #pragma unroll
                     for (int e = 0; e < 4; ++e) if (kg + e < p.K) v[e] = ld_f((const T*)p.x + (size_t)m * p.ldx + kg + e);
@@ -356,18 +363,27 @@ __global__ void __launch_bounds__(DG_THREADS) gemv_fma_kernel(const DenseGemvPar
         y_s[nl][m] = v;
     }
     __syncthreads();
-    dg_epilogue<T>(p, y_s, tid, lane, warp);
+    dg_epilogue<T, EXT>(p, y_s, tid, lane, warp);
 }
 
-template <typename T, int MR>
+template <typename T, int MR, bool EXT>
 static int launch_dg(const DenseGemvParams* p, cudaStream_t s) {
     const int WK = DG_WARPS / (p->rpc >> 2), unit = DG_U * WK * 32 * DgVec<T>::V, cap = 32768 / MR;
     int KC = (p->K + unit - 1) / unit * unit;
     if (KC > cap) KC = cap / unit * unit;
     const size_t smem = (size_t)MR * KC * sizeof(T);
     static SmemOptIn opt;
-    if (int e = opt.ensure((const void*)gemv_fma_kernel<T, MR>, smem)) return e;
-    return launch_pdl(gemv_fma_kernel<T, MR>, dim3((p->N + p->rpc - 1) / p->rpc), dim3(DG_THREADS), smem, s, *p, KC);
+    if (int e = opt.ensure((const void*)gemv_fma_kernel<T, MR, EXT>, smem)) return e;
+    return launch_pdl(gemv_fma_kernel<T, MR, EXT>, dim3((p->N + p->rpc - 1) / p->rpc), dim3(DG_THREADS), smem, s, *p, KC);
+}
+
+template <bool EXT>
+static int launch_dg_rows(const DenseGemvParams* p, cudaStream_t s) {
+    if (p->dt == DT_BF16) return p->rows == 1 ? launch_dg<bf16, 1, EXT>(p, s) : launch_dg<bf16, 2, EXT>(p, s);
+    if (p->rows == 1) return launch_dg<float, 1, EXT>(p, s);
+    if (p->rows == 2) return launch_dg<float, 2, EXT>(p, s);
+    if (p->rows <= 4) return launch_dg<float, 4, EXT>(p, s);
+    return launch_dg<float, 8, EXT>(p, s);
 }
 
 // rpc (outputs per CTA): 8, 16 or 32 in fp32 and for one or two bf16 rows, 16, 32, 64 or 128 for more bf16 rows
@@ -379,17 +395,14 @@ B2_API int b2_gemv_dense(const DenseGemvParams* p, cudaStream_t s) {
     if (p->x ? (p->ldx < p->K || ((uintptr_t)p->x & 15)) : ((!p->pn.h && !p->pn.m) || p->pn.H != p->K)) return cudaErrorInvalidValue;
     if (p->mode == DG_STREAMS && (p->sm.n < 1 || p->sm.n > STREAMS_MAX || !p->sm.x || !p->sm.u || !p->sm.coef)) return cudaErrorInvalidValue;
     if (p->ss_out && (p->N + p->rpc - 1) / p->rpc > p->ss_np) return cudaErrorInvalidValue;
+    const bool ext = dg_extended(*p);
     const bool tc = p->dt == DT_BF16 && (p->mma || p->rows > DG_FMA_ROWS);
     if (tc) {
         if (p->rpc != 16 && p->rpc != 32 && p->rpc != 64 && p->rpc != 128) return cudaErrorInvalidValue;
-        return launch_dm(p, s);
+        return ext ? launch_dm<true>(p, s) : launch_dm<false>(p, s);
     }
     if (p->rpc != 8 && p->rpc != 16 && p->rpc != 32) return cudaErrorInvalidValue;
-    if (p->dt == DT_BF16) return p->rows == 1 ? launch_dg<bf16, 1>(p, s) : launch_dg<bf16, 2>(p, s);
-    if (p->dt != DT_F32) return cudaErrorInvalidValue;
-    if (p->rows == 1) return launch_dg<float, 1>(p, s);
-    if (p->rows == 2) return launch_dg<float, 2>(p, s);
-    if (p->rows <= 4) return launch_dg<float, 4>(p, s);
-    return launch_dg<float, 8>(p, s);
+    if (p->dt != DT_BF16 && p->dt != DT_F32) return cudaErrorInvalidValue;
+    return ext ? launch_dg_rows<true>(p, s) : launch_dg_rows<false>(p, s);
 }
 B2_API int b2_sizeof_dense_gemv_params() { return (int)sizeof(DenseGemvParams); }

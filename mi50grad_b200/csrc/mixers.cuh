@@ -173,10 +173,15 @@ struct MixLayer {
     int gate;                                             // REC_GATE_*
     int out_col;                                          // column of the output row where the recurrence starts
     int exact_weights;                                    // prompt attention: 1 = soft-max weights keep all 24 bits in the
-                                                          // product with V, 0 = they are rounded to bf16
+                                                          // product with V (always so with a softcap), 0 = rounded to bf16
 };
 #define REC_GATE_SILU_NORM 0   // norm(y * silu(z)) in ngroups equal parts
 #define REC_NORM_SIGMOID 1     // norm(y) * sigmoid(z)
+
+static inline bool attn_valid(const MixLayer* l) {
+    return l->H >= 1 && l->G >= 1 && l->H % l->G == 0 && l->d >= 1 && l->dp >= l->d && l->dp <= 256 && !(l->dp & 7) && l->dv >= 1 &&
+           l->vp >= l->dv && l->vp <= 256 && !(l->vp & 7) && l->rot <= l->d && !(l->rot & 1) && l->keep_first >= 0;
+}
 
 struct MixRun {
     const void* proj; int ld_proj; int dt;
