@@ -4,7 +4,7 @@
 #include "mixers.cuh"
 
 // ---------------------------------------------------------------------------
-// many rows of ONE sequence, bf16: grid (64-row tiles, H), four warps of 16 rows
+// many rows of ONE sequence, bf16: grid (H, 64-row tiles), four warps of 16 rows
 // ---------------------------------------------------------------------------
 #define WR_ROWS 64
 #define WR_KEYS 64
@@ -43,7 +43,7 @@ __device__ __forceinline__ float wr_cap(float x, float cap, float e) { return ca
 // TERMS: bf16 terms of a soft-max weight in the product with V (1: the weight rounded to bf16, 3: all of its 24 bits)
 // CAP: capped scores.
 template <int DP, int TERMS, bool CAP>
-__global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, const MixRun R) {
+__global__ void __launch_bounds__(128, 1) window_rows_kernel(const MixLayer L, const MixRun R) {
     constexpr int LD = DP + WR_PAD, NT_O = DP / 8, PPR = DP / 8;
     extern __shared__ __align__(16) unsigned char wrs[];
     bf16* Qs = (bf16*)wrs;                       // [64][LD]
@@ -51,7 +51,8 @@ __global__ void __launch_bounds__(128) window_rows_kernel(const MixLayer L, cons
     bf16* Vb = Kb + 2 * WR_KEYS * LD;            // [2][64][LD]
     pdl_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int row0 = blockIdx.x * WR_ROWS, nrows = min(WR_ROWS, R.n_rows - row0), head = blockIdx.y;
+    // (the tiles that see most keys start first)
+    const int row0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * WR_ROWS, nrows = min(WR_ROWS, R.n_rows - row0), head = blockIdx.x;
     const int kvh = head / (L.H / L.G);
     const RowMeta rm = R.rows[row0];
     const int p0 = rm.pos;                       // positions of the tile: p0 .. p0 + nrows - 1
@@ -200,7 +201,7 @@ static int launch_wr(const MixLayer* l, const MixRun* r, cudaStream_t s) {
     const size_t smem = (size_t)(WR_ROWS + 4 * WR_KEYS) * (DP + WR_PAD) * sizeof(bf16);
     static SmemOptIn opt;
     if (int e = opt.ensure((const void*)window_rows_kernel<DP, TERMS, CAP>, smem)) return e;
-    return launch_pdl(window_rows_kernel<DP, TERMS, CAP>, dim3((r->n_rows + WR_ROWS - 1) / WR_ROWS, l->H), dim3(128), smem, s, *l, *r);
+    return launch_pdl(window_rows_kernel<DP, TERMS, CAP>, dim3(l->H, (r->n_rows + WR_ROWS - 1) / WR_ROWS), dim3(128), smem, s, *l, *r);
 }
 template <int TERMS, bool CAP>
 static int launch_wr_t(const MixLayer* l, const MixRun* r, cudaStream_t s) {
