@@ -334,8 +334,8 @@ class SSDSpec:
 
 @dataclass(frozen=True)
 class LightningSpec:
-    """Linear attention S <- decay_h S + k v^T, o = S^T q with a constant decay per head; every head has its
-    own q and k (of size `state`) and v (of size `vdim`)."""
+    """Linear attention over a state that fades by a constant factor per head and token; every head has its own
+    q and k (of size `state`) and v (of size `vdim`)."""
     heads: int
     state: int
     vdim: int

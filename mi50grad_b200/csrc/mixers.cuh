@@ -44,9 +44,8 @@ struct PostNorm {
 
 // ---------------------------------------------------------------------------
 // Hyper-connections: a row has `n` residual streams x_0 .. x_(n-1).  Between two sublayers
-//     x_t <- sum_s mix[s][t] x_s + out[t] * y          (y: output of the sublayer before)
-//     u    = sum_s in[s] x_s                           (input of the next sublayer, before its norm)
-// coef: mix [n][n] | out [n] | in [n].
+//     X' = Mix^T X + Out y^T,   u = In^T X'     (X: the streams as rows; y: output of the sublayer before, u: input
+// of the next one, before its norm).  coef: Mix [n][n] | Out [n] | In [n].
 // ---------------------------------------------------------------------------
 struct StreamMix {
     float* x;                // [rows][n][H], updated in place

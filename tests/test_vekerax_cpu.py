@@ -126,7 +126,7 @@ def test_recurrence_and_gate_by_hand():
 
 
 def test_streams_by_hand():
-    # mixing weights are indexed [from, to]
+    # row of M: where a part comes from; column: where it goes
     xs = torch.tensor([1.0, 10.0]).reshape(2, 1, 1)
     M, b = torch.tensor([[1.0, 2.0], [3.0, 4.0]]), torch.tensor([0.5, -1.0])
     new = O.streams_out(xs, M, b, 0.1, torch.tensor([[20.0]]))

@@ -70,8 +70,8 @@ def attention_mixer(c, eps, W, p, x, cache):
 
 
 def decayed_outer_recurrence(q, k, v, decay, S):
-    """S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; q, k [n, heads, dim], v [n, heads, vdim],
-    S [heads, dim, vdim].  Returns (o [n, heads, vdim], last state)."""
+    """Every token fades a head's matrix by the head's constant, adds the outer product of its key and value, and
+    reads the result with its query; q, k [n, heads, dim], v [n, heads, vdim], S [heads, dim, vdim].  Returns (o [n, heads, vdim], last state)."""
     n, H, _ = q.shape
     o = torch.zeros_like(v)
     S = S.clone()
@@ -100,12 +100,12 @@ def lightning_mixer(c, eps, W, p, x, state):
 
 
 def streams_in(xs, a):
-    """xs [streams, n, width] -> sum_s a[s] x_s"""
+    """xs [streams, n, width] -> their sum weighted by a"""
     return (a.to(xs.dtype)[:, None, None] * xs).sum(0)
 
 
 def streams_out(xs, M, b, m, y):
-    """x_t <- sum_s M[s, t] x_s + m b[t] y"""
+    """New streams: column t of M weighs the old ones, plus y times m b[t]."""
     new = torch.zeros_like(xs)
     for t in range(xs.shape[0]):
         for s in range(xs.shape[0]):
